@@ -1,5 +1,5 @@
-from .cache import PAGE_SIZE, Cache, CacheEntries, CacheEntry, CacheSpec, KVGroup, KVSpec, StateGroup, StateSpec
+from .cache import PAGE_SIZE, Cache, CacheEntries, CacheEntry, CacheSpec, KVGroup, KVSpec, StateGroup, StateSpec, shared_spec
 from .pages import CacheError, CacheFull, PagePool, SlotTable
 
 __all__ = ["PAGE_SIZE", "Cache", "CacheEntries", "CacheEntry", "CacheSpec", "KVGroup", "KVSpec", "StateGroup", "StateSpec",
-           "CacheError", "CacheFull", "PagePool", "SlotTable"]
+           "shared_spec", "CacheError", "CacheFull", "PagePool", "SlotTable"]

@@ -18,6 +18,7 @@ Layers whose needs are equal form a *group* with storage of its own:
 * a group that sees a chunk of C keys (position p sees the keys from
   ``p - p % C`` on) holds the same ring as a window of C: a chunk never spans
   more places than the ring has;
+* an entry that other schedule entries read (``shared_spec``) keeps what the widest of their masks sees;
 * a windowed group that also keeps a sequence's first F keys visible for good
   (``keep_first``) holds ``round_up(F, page_size)`` places ahead of the ring:
   position p lives at place p below that bound and at
@@ -81,6 +82,22 @@ def kept_span(spec: KVSpec) -> Optional[int]:
     """How many of the newest keys a sequence has to keep (None: all of them)."""
     spans = [s for s in (spec.window, spec.chunk) if s]
     return min(spans) if spans else None
+
+
+def shared_spec(own: KVSpec, readers: Sequence[KVSpec]) -> KVSpec:
+    """What an entry has to keep so that its own mask and those of the entries that read its keys and values find
+    all they see: the widest span of the newest keys (all keys if one of them sees all), the most kept first keys."""
+    for r in readers:
+        if not isinstance(own, KVSpec) or not isinstance(r, KVSpec) or \
+                (r.n_kv, r.head_dim, r.values, r.v_dim) != (own.n_kv, own.head_dim, own.values, own.v_dim):
+            raise CacheError(f"an entry that keeps {own!r} cannot be read by one that needs {r!r}")
+    everyone = [own, *readers]
+    spans = [kept_span(s) for s in everyone]
+    if all(s == own for s in readers) or (kept_span(own) is None and not own.chunk):
+        return own
+    if None in spans:
+        return dataclasses.replace(own, window=None, chunk=None, keep_first=0)
+    return dataclasses.replace(own, window=max(spans), chunk=None, keep_first=max(s.keep_first for s in everyone))
 
 
 class KVGroup:

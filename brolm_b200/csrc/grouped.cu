@@ -30,11 +30,13 @@ constexpr int GBM = 64, GBN = 64;
 // mode ROUTE_LOGISTIC: the weight of a chosen expert is the logistic function of its score.
 // mode ROUTE_SOFTMAX: s = softmax(z) over all experts; the choice goes by s + corr (a learned number per expert
 // that takes no part in the weights); the weights are the chosen s over their sum (+ 1e-20).
+// mode ROUTE_CHOSEN: the choice goes by z itself and the weights are the softmax over the chosen scores alone.
+// In every mode `bias` (a number per expert, or null) is added to z first and is part of the score.
 // The softmax mode's further options (RouteOpts): the experts form `groups` equal groups of neighbours, a group's
 // score is the largest s + corr in it, and only experts of the `keep` best groups (ties: the lower group) can be
 // chosen; `renorm` 0 leaves the chosen s as they are instead of dividing by their sum; `wscale` multiplies the
 // weights at the end.
-enum : int { ROUTE_LOGISTIC = 0, ROUTE_SOFTMAX = 1 };
+enum : int { ROUTE_LOGISTIC = 0, ROUTE_SOFTMAX = 1, ROUTE_CHOSEN = 2 };
 
 struct RouteOpts {
     int groups, keep, renorm;
@@ -43,7 +45,11 @@ struct RouteOpts {
 
 __device__ __forceinline__ void pick_top(float* zr, int E, int top, int t, int lane, int32_t* __restrict__ ids,
                                          float* __restrict__ wts, int mode, const float* __restrict__ corr,
-                                         RouteOpts ro) {
+                                         RouteOpts ro, const float* __restrict__ bias) {
+    if (bias) {
+        for (int e = lane; e < E; e += 32) zr[e] += bias[e];
+        __syncwarp();
+    }
     if (mode == ROUTE_SOFTMAX) {
         float m = -INFINITY;
         for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
@@ -115,6 +121,7 @@ __device__ __forceinline__ void pick_top(float* zr, int E, int top, int t, int l
         }
         return;
     }
+    float first = 0.0f, total = 0.0f;                  // ROUTE_CHOSEN: the largest score, the sum of the exponentials
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = 0x7fffffff;
@@ -131,18 +138,28 @@ __device__ __forceinline__ void pick_top(float* zr, int E, int top, int t, int l
         if (at >= E) at = 0;                       // (every score was -inf or NaN)
         if (lane == 0) {
             ids[(size_t)t * top + k] = at;
-            wts[(size_t)t * top + k] = 1.0f / (1.0f + expf(-best));
+            if (mode == ROUTE_CHOSEN) {
+                if (k == 0) first = best;
+                const float w = expf(best - first);
+                wts[(size_t)t * top + k] = w;
+                total += w;
+            } else {
+                wts[(size_t)t * top + k] = 1.0f / (1.0f + expf(-best));
+            }
             zr[at] = -INFINITY;
         }
         __syncwarp();
     }
+    if (mode == ROUTE_CHOSEN && lane == 0)
+        for (int k = 0; k < top; ++k) wts[(size_t)t * top + k] /= total;
 }
 
 template <typename T, int RT>
 __global__ void __launch_bounds__(RT == 1 ? 1024 : 256) route_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ wr,
                                                     int E, int D, int top, int tokens, int vec,
                                                     int32_t* __restrict__ ids, float* __restrict__ wts, int mode,
-                                                    const float* __restrict__ corr, RouteOpts ro) {
+                                                    const float* __restrict__ corr, RouteOpts ro,
+                                                    const float* __restrict__ bias) {
     extern __shared__ float z[];                       // [RT][E]
     const int t0 = blockIdx.x * RT;
     const int nt = min(RT, tokens - t0);
@@ -217,14 +234,15 @@ __global__ void __launch_bounds__(RT == 1 ? 1024 : 256) route_kernel(const T* __
         }
     }
     __syncthreads();
-    for (int r = warp; r < nt; r += nwarps) pick_top(z + r * E, E, top, t0 + r, lane, ids, wts, mode, corr, ro);
+    for (int r = warp; r < nt; r += nwarps) pick_top(z + r * E, E, top, t0 + r, lane, ids, wts, mode, corr, ro, bias);
 }
 
 // The choice alone, for scores that a matrix product left in memory: z [tokens, E] float (ldz between rows).
 // A block takes eight tokens, a warp one.
 __global__ void __launch_bounds__(256) route_pick_kernel(const float* __restrict__ zs, long ldz, int E, int top, int tokens,
                                                          int32_t* __restrict__ ids, float* __restrict__ wts, int mode,
-                                                         const float* __restrict__ corr, RouteOpts ro) {
+                                                         const float* __restrict__ corr, RouteOpts ro,
+                                                         const float* __restrict__ bias) {
     extern __shared__ float z[];                       // [8][E]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * 8 + warp;
@@ -232,7 +250,7 @@ __global__ void __launch_bounds__(256) route_pick_kernel(const float* __restrict
     float* zr = z + warp * E;
     for (int e = lane; e < E; e += 32) zr[e] = zs[(size_t)t * ldz + e];
     __syncwarp();
-    pick_top(zr, E, top, t, lane, ids, wts, mode, corr, ro);
+    pick_top(zr, E, top, t, lane, ids, wts, mode, corr, ro, bias);
 }
 
 // ---------------------------------------------------------------------------
@@ -703,6 +721,7 @@ int launch_grouped(int dtype, GroupedArgs& g, int row_tiles, bool few, cudaStrea
 // ids [tokens, top] int32 and wts [tokens, top] float: the chosen experts of every token, best first.
 // mode 0: the weights are the logistic function of the chosen scores; mode 1: softmax over all experts, the choice
 // by softmax + corr (float [experts] or null), the weights the chosen softmax values over their sum.
+// mode 2: the choice by z, the weights the softmax over the chosen z alone.  bias (float [experts] or null) is added to z.
 // groups, keep, renorm, wscale: the softmax mode's options (see RouteOpts); 1, 1, 1, 1.0 are the plain router.
 static inline bool route_opts_ok(int experts, int top, int groups, int keep) {
     return groups >= 1 && keep >= 1 && keep <= groups && experts % groups == 0 && top <= keep * (experts / groups);
@@ -710,7 +729,7 @@ static inline bool route_opts_ok(int experts, int top, int groups, int keep) {
 
 BROLM_API int brolm_route_topk(int dtype, const void* x, long ldx, const void* wr, int tokens, int experts, int width,
                                int top, void* ids, void* wts, int mode, const void* corr, int groups, int keep,
-                               int renorm, float wscale, cudaStream_t stream) {
+                               int renorm, float wscale, const void* bias, cudaStream_t stream) {
     if (tokens <= 0) return BROLM_OK;
     if (experts <= 0 || top <= 0 || top > experts || width <= 0) return BROLM_ERR_BAD_SIZE;
     if (!route_opts_ok(experts, top, groups, keep)) return BROLM_ERR_BAD_SIZE;
@@ -723,7 +742,8 @@ BROLM_API int brolm_route_topk(int dtype, const void* x, long ldx, const void* w
     const int blocks = (tokens + rt - 1) / rt;
 #define BROLM_ROUTE(T, RT)                                                                                        \
     route_kernel<T, RT><<<blocks, RT == 1 ? 1024 : 256, smem, stream>>>((const T*)x, ldx, (const T*)wr, experts, width, top, tokens, \
-                                                       vec, (int32_t*)ids, (float*)wts, mode, (const float*)corr, ro)
+                                                       vec, (int32_t*)ids, (float*)wts, mode, (const float*)corr, ro,    \
+                                                       (const float*)bias)
     if (dtype == BROLM_F32) {
         if (many) BROLM_ROUTE(float, 4); else BROLM_ROUTE(float, 1);
     } else if (dtype == BROLM_BF16) {
@@ -738,14 +758,15 @@ BROLM_API int brolm_route_topk(int dtype, const void* x, long ldx, const void* w
 // The same choice from scores already in memory: z [tokens, experts] float, ldz floats between rows.
 BROLM_API int brolm_route_pick(const void* z, long ldz, int tokens, int experts, int top, void* ids, void* wts,
                                int mode, const void* corr, int groups, int keep, int renorm, float wscale,
-                               cudaStream_t stream) {
+                               const void* bias, cudaStream_t stream) {
     if (tokens <= 0) return BROLM_OK;
     if (experts <= 0 || top <= 0 || top > experts) return BROLM_ERR_BAD_SIZE;
     if (!route_opts_ok(experts, top, groups, keep)) return BROLM_ERR_BAD_SIZE;
     const RouteOpts ro = {groups, keep, renorm, wscale};
     if (experts > 1024) return BROLM_ERR_TOO_LARGE;          // (eight rows of scores in the default shared memory)
     route_pick_kernel<<<(tokens + 7) / 8, 256, (size_t)8 * experts * sizeof(float), stream>>>(
-        (const float*)z, ldz, experts, top, tokens, (int32_t*)ids, (float*)wts, mode, (const float*)corr, ro);
+        (const float*)z, ldz, experts, top, tokens, (int32_t*)ids, (float*)wts, mode, (const float*)corr, ro,
+        (const float*)bias);
     return launch_status();
 }
 

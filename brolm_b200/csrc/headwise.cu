@@ -14,6 +14,7 @@
 //       its own values, as they are before any mixing, for the later ones);
 //     * the result in the step's element type, rounded once, into the packed row and into the cache pages
 //       (k rows of hd, value rows of vd; cache_rows[t] = page * page_size + place, negative: not kept).
+//   n_kv may be 0: a row of queries alone (a layer that reads another layer's keys and values).
 //   A negative position marks a padding row, which is left untouched.
 //
 // heads_mix: what lies between an attention whose heads' weights are mixed after the softmax and the output product.
@@ -258,7 +259,8 @@ BROLM_API int brolm_qkv_finish(const void* proj, int x_dtype, int n_parts, long 
                                const void* cache_rows, int page_size, int tokens, const void* q_gain, const void* k_gain,
                                cudaStream_t stream) {
     if (tokens <= 0) return BROLM_OK;
-    if (n_q <= 0 || n_kv <= 0 || hd <= 0 || vd <= 0 || n_parts < 1) return BROLM_ERR_BAD_SIZE;
+    if (n_q <= 0 || n_kv < 0 || hd <= 0 || vd <= 0 || n_parts < 1) return BROLM_ERR_BAD_SIZE;
+    if (n_kv == 0 && (k_pages || v_pages)) return BROLM_ERR_BAD_SIZE;
     if (cos_sin && (rot <= 0 || rot % 2 || rot > hd || pairing < 0 || pairing > 1)) return BROLM_ERR_BAD_SIZE;
     if (n_parts > 1 && x_dtype != BROLM_F32) return BROLM_ERR_BAD_DTYPE;
     const size_t smem = (size_t)((n_q + n_kv) * hd + n_kv * vd) * sizeof(float);

@@ -18,6 +18,11 @@
 // then folded across its DS lanes by shuffles, sixteen tokens at once.  Sequential in the tokens: the order of the
 // additions of a token's result does not depend on how the sequence was cut into steps, only (through DS) on the
 // launch's size.
+//
+// q and k may be rotated by their token's position (pairs (i, i + rot/2) of a head's first `rot` entries, cos and sin
+// from a table) and k scaled by a constant before they enter the recurrence, in float.  Single tokens: the scan does it
+// on the staged rows (ROT variants of the kernel; a launch without them carries none of it).  A prompt: rotate_heads,
+// in place and once, since the blocks of a head would each do it anew.
 #include <type_traits>
 
 #include "common.cuh"
@@ -41,6 +46,9 @@ struct ScanArgs {
     int ds;                   // lanes per value column (a power of two, at most 32)
     int vec;                  // float rows: every run of q, k and v starts at a multiple of 16 bytes
     int early;                // a step of single tokens: takes part in programmatic launch
+    const float* cos_sin;     // ROT: [positions][rot / 2][2], or null (k_scale alone)
+    int rot;
+    float k_scale;
 };
 
 constexpr int SCAN_TC = 16;
@@ -63,7 +71,8 @@ __device__ __forceinline__ void scan_cp16(float* dst, const float* src) {
 // are read, one buffer.
 // DSC > 0: the lanes per column are known to the compiler and NJ * DSC float4 are exactly a row of d (no padding, no
 // bounds in the inner loop, every offset a constant); DSC = 0: any d, lanes per column from the launch.
-template <typename X, int NJ, int DSC>
+// ROT: rotate the staged q and k and scale k (float rows only).
+template <typename X, int NJ, int DSC, bool ROT>
 __global__ void __launch_bounds__(128) decay_scan_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float sm[];
     if (a.early) pdl_trigger();
@@ -88,6 +97,16 @@ __global__ void __launch_bounds__(128) decay_scan_kernel(ScanArgs a) {
         float4 s4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (live && f < dp4) s4 = *reinterpret_cast<const float4*>(st + 4 * f);
         S[4 * j] = s4.x; S[4 * j + 1] = s4.y; S[4 * j + 2] = s4.z; S[4 * j + 3] = s4.w;
+    }
+    // the table's entries of a thread's first pair are on their way before the rows of this step are there
+    const int half = a.rot >> 1, pos0 = kv_len - q_len;
+    float c0 = 1.0f, s0 = 0.0f;
+    if constexpr (ROT) {
+        if ((int)threadIdx.x < min(SCAN_TC, q_len) * half) {
+            const int tt = threadIdx.x / half;
+            const float2 e = reinterpret_cast<const float2*>(a.cos_sin)[(size_t)(pos0 + tt) * half + (threadIdx.x - tt * half)];
+            c0 = e.x; s0 = e.y;
+        }
     }
     if (ASYNC) {
         // the padding of d to a multiple of four, and value columns beyond dv, stay zero in both buffers
@@ -154,6 +173,29 @@ __global__ void __launch_bounds__(128) decay_scan_kernel(ScanArgs a) {
                                                         : 2 * SCAN_TC * dp + (idx - 2 * n_tok * dp);
                     const float x = sq[at];
                     sq[at] = x / (1.0f + expf(-x));
+                }
+                __syncthreads();
+            }
+            if constexpr (ROT) {
+                for (int idx = threadIdx.x; idx < n_tok * half; idx += 128) {
+                    const int tt = idx / half, i = idx - tt * half;
+                    float c = c0, s = s0;
+                    if (kc > 0 || idx != (int)threadIdx.x) {
+                        const float2 e = reinterpret_cast<const float2*>(a.cos_sin)[(size_t)(pos0 + t0 + tt) * half + i];
+                        c = e.x; s = e.y;
+                    }
+                    float* qr = sq + tt * dp + i;
+                    float* kr = sk + tt * dp + i;
+                    const float qu = qr[0], qw = qr[half], ku = kr[0], kw = kr[half];
+                    qr[0] = qu * c - qw * s;
+                    qr[half] = qw * c + qu * s;
+                    kr[0] = (ku * c - kw * s) * a.k_scale;
+                    kr[half] = (kw * c + ku * s) * a.k_scale;
+                }
+                const int rest = a.d - a.rot;
+                for (int idx = threadIdx.x; idx < n_tok * rest; idx += 128) {
+                    const int tt = idx / rest;
+                    sk[tt * dp + a.rot + idx - tt * rest] *= a.k_scale;
                 }
                 __syncthreads();
             }
@@ -237,7 +279,6 @@ __global__ void __launch_bounds__(128) decay_scan_kernel(ScanArgs a) {
             pv[0] += __shfl_xor_sync(0xffffffffu, pv[0], o);
             writer = writer && (ds & 1) == 0;
         }
-#pragma unroll
         float* orow = a.out + (size_t)(q0 + t0 + first) * a.ldo + (size_t)h * a.dv + v;
 #pragma unroll
         for (int i = 0; i < SCAN_TC; ++i)
@@ -253,17 +294,25 @@ __global__ void __launch_bounds__(128) decay_scan_kernel(ScanArgs a) {
     }
 }
 
-template <typename X, int NJ, int DSC>
-int launch_scan_as(const ScanArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+template <typename X, int NJ, int DSC, bool ROT>
+int launch_scan_rot(const ScanArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
     static size_t allowed = 0;
     if (smem > 48 * 1024 && smem > allowed) {
-        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<X, NJ, DSC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<X, NJ, DSC, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         allowed = smem;
     }
     // a prompt's scan runs long on few warps: plain stream order, so that its blocks spread evenly over the SMs
-    if (!a.early) return launch_in_order(decay_scan_kernel<X, NJ, DSC>, grid, dim3(128), smem, stream, a);
-    return launch_pdl(decay_scan_kernel<X, NJ, DSC>, grid, dim3(128), smem, stream, a);
+    if (!a.early) return launch_in_order(decay_scan_kernel<X, NJ, DSC, ROT>, grid, dim3(128), smem, stream, a);
+    return launch_pdl(decay_scan_kernel<X, NJ, DSC, ROT>, grid, dim3(128), smem, stream, a);
+}
+
+template <typename X, int NJ, int DSC>
+int launch_scan_as(const ScanArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
+    if constexpr (sizeof(X) == 4) {
+        if (a.rot > 0 || a.k_scale != 1.0f) return launch_scan_rot<X, NJ, DSC, true>(a, grid, smem, stream);
+    }
+    return launch_scan_rot<X, NJ, DSC, false>(a, grid, smem, stream);
 }
 
 template <typename X>
@@ -303,13 +352,81 @@ int launch_scan(const ScanArgs& a0, int batch, int max_q_len, cudaStream_t strea
     return launch_scan_as<X, 4, 0>(a, grid, smem, stream);
 }
 
+// q and k of a prompt's float rows, in place: every head's first `rot` entries rotated by the token's position, k scaled.
+// V neighbours of a pair's halves (and of the entries that pass unrotated) a thread; grid (tokens, pieces of a row).
+template <int V>
+__global__ void __launch_bounds__(256) rotate_heads_kernel(float* __restrict__ rows, long ld, int q_off, int k_off, int heads, int d,
+                                                           const int32_t* __restrict__ positions,
+                                                           const float* __restrict__ cos_sin, int rot, float k_scale) {
+    pdl_trigger();
+    const int t = blockIdx.x, pos = positions[t];
+    pdl_wait();
+    if (pos < 0) return;                               // a padding row
+    const int half = rot >> 1, pairs = half / V, items = pairs + (d - rot) / V;
+    float* row = rows + (size_t)t * ld;
+    const float* cs = cos_sin ? cos_sin + (size_t)pos * half * 2 : nullptr;
+    for (int idx = blockIdx.y * blockDim.x + threadIdx.x; idx < 2 * heads * items; idx += gridDim.y * blockDim.x) {
+        const int h2 = idx / items, it = idx - h2 * items;
+        const bool is_k = h2 >= heads;
+        float* x = row + (is_k ? k_off + (h2 - heads) * d : q_off + h2 * d);
+        const float f = is_k ? k_scale : 1.0f;
+        if (it >= pairs) {
+            if (!is_k || f == 1.0f) continue;
+            float* p = x + rot + (it - pairs) * V;
+            if constexpr (V == 4) {
+                float4 v = *reinterpret_cast<float4*>(p);
+                v.x *= f; v.y *= f; v.z *= f; v.w *= f;
+                *reinterpret_cast<float4*>(p) = v;
+            } else {
+                *p *= f;
+            }
+            continue;
+        }
+        const int i = it * V;
+        if constexpr (V == 4) {
+            const float4 u = *reinterpret_cast<float4*>(x + i), w = *reinterpret_cast<float4*>(x + half + i);
+            const float4 e0 = *reinterpret_cast<const float4*>(cs + 2 * i), e1 = *reinterpret_cast<const float4*>(cs + 2 * i + 4);
+            float4 a, b;
+            a.x = (u.x * e0.x - w.x * e0.y) * f; b.x = (w.x * e0.x + u.x * e0.y) * f;
+            a.y = (u.y * e0.z - w.y * e0.w) * f; b.y = (w.y * e0.z + u.y * e0.w) * f;
+            a.z = (u.z * e1.x - w.z * e1.y) * f; b.z = (w.z * e1.x + u.z * e1.y) * f;
+            a.w = (u.w * e1.z - w.w * e1.w) * f; b.w = (w.w * e1.z + u.w * e1.w) * f;
+            *reinterpret_cast<float4*>(x + i) = a;
+            *reinterpret_cast<float4*>(x + half + i) = b;
+        } else {
+            const float u = x[i], w = x[half + i], c = cs[2 * i], s = cs[2 * i + 1];
+            x[i] = (u * c - w * s) * f;
+            x[half + i] = (w * c + u * s) * f;
+        }
+    }
+}
+
 }  // namespace
+
+// rows [tokens][ld] float, changed in place: heads of d at q_off and k_off; cos_sin null: no rotation (rot 0).
+BROLM_API int brolm_rotate_heads(void* rows, long ld, int q_off, int k_off, int heads, int d, const void* positions,
+                                 const void* cos_sin, int rot, float k_scale, int tokens, cudaStream_t stream) {
+    if (tokens <= 0) return BROLM_OK;
+    if (heads <= 0 || d <= 0 || rot < 0 || rot % 2 || rot > d || (rot > 0) != (cos_sin != nullptr)) return BROLM_ERR_BAD_SIZE;
+    const bool four = d % 4 == 0 && rot % 8 == 0 && ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
+                      ((uintptr_t)rows & 15) == 0 && ((uintptr_t)cos_sin & 15) == 0;
+    const int v = four ? 4 : 1;
+    const int items = 2 * heads * (rot / 2 / v + (d - rot) / v);
+    int by = (items + 255) / 256;
+    if (by > 64) by = 64;
+    dim3 grid(tokens, by);
+    if (four)
+        return launch_pdl(rotate_heads_kernel<4>, grid, dim3(256), 0, stream, (float*)rows, ld, q_off, k_off, heads, d,
+                          (const int32_t*)positions, (const float*)cos_sin, rot, k_scale);
+    return launch_pdl(rotate_heads_kernel<1>, grid, dim3(256), 0, stream, (float*)rows, ld, q_off, k_off, heads, d,
+                      (const int32_t*)positions, (const float*)cos_sin, rot, k_scale);
+}
 
 // The state row of a sequence holds heads * dv * round_up(d, 4) floats for this mixer, from `state` on.
 BROLM_API int brolm_decay_scan(const void* qkv, int x_dtype, long ld, int q_off, int k_off, int v_off, int heads, int d,
                                int dv, int act, const void* decay_m1, const void* cu_q, const void* kv_len,
                                const void* slots, void* state, long state_stride, void* out, long ldo, int batch,
-                               int max_q_len, cudaStream_t stream) {
+                               int max_q_len, const void* cos_sin, int rot, float k_scale, cudaStream_t stream) {
     if (batch <= 0) return BROLM_OK;
     if (heads <= 0 || d <= 0 || dv <= 0 || act < 0 || act > 1) return BROLM_ERR_BAD_SIZE;
     if (heads > 65535 || batch > 65535) return BROLM_ERR_TOO_LARGE;
@@ -320,6 +437,9 @@ BROLM_API int brolm_decay_scan(const void* qkv, int x_dtype, long ld, int q_off,
     a.decay_m1 = (const float*)decay_m1;
     a.cu_q = (const int32_t*)cu_q; a.kv_len = (const int32_t*)kv_len; a.slots = (const int32_t*)slots;
     a.state = (float*)state; a.state_stride = state_stride; a.out = (float*)out; a.ldo = ldo; a.ds = 1; a.early = 0;
+    if (rot < 0 || rot % 2 || rot > d || (rot > 0) != (cos_sin != nullptr)) return BROLM_ERR_BAD_SIZE;
+    if ((rot > 0 || k_scale != 1.0f) && x_dtype != BROLM_F32) return BROLM_ERR_BAD_DTYPE;
+    a.cos_sin = (const float*)cos_sin; a.rot = rot; a.k_scale = k_scale;
     a.vec = x_dtype == BROLM_F32 && d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
             v_off % 4 == 0 && ((uintptr_t)qkv & 15) == 0;
     if (x_dtype == BROLM_F32) return launch_scan<float>(a, batch, max_q_len, stream);

@@ -10,6 +10,8 @@
 //   experts_combine out = sum over a token's choices of weight * (expert's result | the token's own
 //                   row for an identity expert) + the shared expert's result, the latter times
 //                   sigmoid(w . x) when a gate row w is given
+//   head_norm_gate     out = (every head of y divided by its own rms, times a gain if there is one) * gate(z), the gate
+//                      being silu or sigmoid
 //   norm_sigmoid_gate  out = (y / rms(y) * gain, or y itself without a gain) * sigmoid(z)
 //
 // Inputs are float or bfloat16, outputs as asked for.  One block per token (row); a row's result
@@ -297,7 +299,98 @@ __global__ void __launch_bounds__(256) norm_sigmoid_gate_kernel(const Y* __restr
     }
 }
 
+// out[t, h * hd + e] = y[t, h * hd + e] * rsqrt(mean over the head of y^2 + eps) * (w or 1) * gate(z[t, h * hd + e]);
+// gate: 0 silu, 1 sigmoid.  A warp per (token, head).  V = 4: rows, heads and addresses in steps of 16 bytes (8 for a
+// bfloat16 result), the head kept in registers up to NREG pieces a lane; V = 1: anything, read twice.
+__device__ __forceinline__ float gate_of(float z, int gate) {
+    const float s = 1.0f / (1.0f + expf(-z));
+    return gate == 0 ? z * s : s;
+}
+
+__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(bf16* p, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 u;
+    u.x = *reinterpret_cast<uint32_t*>(&a);
+    u.y = *reinterpret_cast<uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = u;
+}
+
+template <typename O, int V>
+__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z,
+                                                             long ldz, const float* __restrict__ w, float eps, int heads, int hd,
+                                                             int gate, O* __restrict__ out, long ldo, int tokens) {
+    constexpr int NREG = 4;
+    pdl_trigger();
+    const int lane = threadIdx.x & 31;
+    const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    pdl_wait();
+    if (unit >= (long long)tokens * heads) return;
+    const int t = (int)(unit / heads), h = (int)(unit - (long long)t * heads);
+    const float* yr = y + (size_t)t * ldy + (size_t)h * hd;
+    const float* zr = z + (size_t)t * ldz + (size_t)h * hd;
+    const float* wr = w ? w + (size_t)h * hd : nullptr;
+    O* orow = out + (size_t)t * ldo + (size_t)h * hd;
+    float ss = 0.0f;
+    if constexpr (V == 4) {
+        float4 v[NREG], g[NREG];
+#pragma unroll
+        for (int j = 0; j < NREG; ++j) {
+            const int e = (j * 32 + lane) * 4;
+            if (e < hd) {
+                v[j] = *reinterpret_cast<const float4*>(yr + e);
+                g[j] = *reinterpret_cast<const float4*>(zr + e);
+                ss += (v[j].x * v[j].x + v[j].y * v[j].y) + (v[j].z * v[j].z + v[j].w * v[j].w);
+            }
+        }
+        const float inv = rsqrtf(warp_sum(ss) / (float)hd + eps);
+#pragma unroll
+        for (int j = 0; j < NREG; ++j) {
+            const int e = (j * 32 + lane) * 4;
+            if (e < hd) {
+                float4 r = make_float4(v[j].x * inv, v[j].y * inv, v[j].z * inv, v[j].w * inv);
+                if (wr) { r.x *= wr[e]; r.y *= wr[e + 1]; r.z *= wr[e + 2]; r.w *= wr[e + 3]; }
+                r.x *= gate_of(g[j].x, gate); r.y *= gate_of(g[j].y, gate);
+                r.z *= gate_of(g[j].z, gate); r.w *= gate_of(g[j].w, gate);
+                store_four(orow + e, r);
+            }
+        }
+    } else {
+        for (int e = lane; e < hd; e += 32) ss = fmaf(yr[e], yr[e], ss);
+        const float inv = rsqrtf(warp_sum(ss) / (float)hd + eps);
+        for (int e = lane; e < hd; e += 32) {
+            float r = yr[e] * inv;
+            if (wr) r *= wr[e];
+            orow[e] = from_float<O>(r * gate_of(zr[e], gate));
+        }
+    }
+}
+
 }  // namespace
+
+// y, z and the gain w (null: none; heads * hd numbers) are float, the result float or bfloat16.
+BROLM_API int brolm_head_norm_gate(const void* y, long ldy, const void* z, long ldz, const void* w, float eps, int heads, int hd,
+                                   int gate, void* out, int out_dtype, long ldo, int tokens, cudaStream_t stream) {
+    if (tokens <= 0) return BROLM_OK;
+    if (heads <= 0 || hd <= 0 || gate < 0 || gate > 1) return BROLM_ERR_BAD_SIZE;
+    const long long units = (long long)tokens * heads;
+    if ((units + 7) / 8 > 0x7fffffff) return BROLM_ERR_TOO_LARGE;
+    const bool four = hd % 4 == 0 && hd <= 512 && ldy % 4 == 0 && ldz % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)y & 15) == 0 &&
+                      ((uintptr_t)z & 15) == 0 && ((uintptr_t)out & 15) == 0;
+    dim3 grid((unsigned)((units + 7) / 8));
+#define BROLM_HN(O, V) return launch_pdl(head_norm_gate_kernel<O, V>, grid, dim3(256), 0, stream, (const float*)y, ldy,   \
+                                         (const float*)z, ldz, (const float*)w, eps, heads, hd, gate, (O*)out, ldo, tokens)
+    if (out_dtype == BROLM_F32) {
+        if (four) BROLM_HN(float, 4);
+        BROLM_HN(float, 1);
+    }
+    if (out_dtype == BROLM_BF16) {
+        if (four) BROLM_HN(bf16, 4);
+        BROLM_HN(bf16, 1);
+    }
+#undef BROLM_HN
+    return BROLM_ERR_BAD_DTYPE;
+}
 
 BROLM_API int brolm_cast(const void* x, int x_dtype, void* out, int out_dtype, long long n, cudaStream_t stream) {
     if (n <= 0) return BROLM_OK;

@@ -13,7 +13,7 @@ from typing import Optional
 import torch
 
 from .. import kernels
-from ..cache import Cache
+from ..cache import Cache, shared_spec
 from ..config import ModelConfig, architecture_of, load_config
 from ..parts import ModelLayout, Part, PartSpec, linear, part_class
 from ..weights import Expected, WeightsError, load_from_folder, load_from_tensors, random_tensors, write_model_folder
@@ -141,9 +141,16 @@ class DecoderModel:
 
     # cache ----------------------------------------------------------------
     def cache_specs(self) -> list:
+        sched = self.layout.schedule
         specs = []
-        for call in self.layout.schedule:
-            specs.append(self.blocks[call.block].cache_spec() if call.cache_of is None else None)
+        for i, call in enumerate(sched):
+            if call.cache_of is not None:
+                specs.append(None)
+                continue
+            own = self.blocks[call.block].cache_spec()
+            # an entry that later ones read keeps what the widest of their masks sees
+            readers = [self.blocks[c.block].cache_spec() for c in sched if c.cache_of == i]
+            specs.append(shared_spec(own, readers) if readers else own)
         return specs
 
     def new_cache(self, max_tokens: int, max_slots: Optional[int] = None, max_seq_len: Optional[int] = None) -> Cache:

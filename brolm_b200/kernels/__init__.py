@@ -282,10 +282,12 @@ def latent_rows(proj: torch.Tensor, q_cols: int, positions: torch.Tensor, cos_si
              _ptr(pages), _ptr(cache_rows) if pages is not None else None, proj.shape[0], _stream()), "latent_rows")
 
 
-ROUTE_MODES = {"logistic": 0, "softmax": 1}
+ROUTE_MODES = {"logistic": 0, "softmax": 1, "softmax_chosen": 2}
 
 
-def _check_route(mode: str, correction: Optional[torch.Tensor], experts: int) -> None:
+def _check_route(mode: str, correction: Optional[torch.Tensor], experts: int, bias: Optional[torch.Tensor] = None) -> None:
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == experts
     if mode not in ROUTE_MODES:
         raise KernelError(f"router: unknown mode '{mode}' (known: {sorted(ROUTE_MODES)})")
     if correction is not None:
@@ -303,37 +305,39 @@ def _route_opts(mode: str, experts: int, top: int, groups: int, keep: int, renor
 
 def route_topk(x: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor,
                mode: str = "logistic", correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1,
-               renorm: bool = True, scale: float = 1.0) -> None:
+               renorm: bool = True, scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """ids, weights [tokens, top]: the ``top`` experts with the largest score, best first (ties: the lower index).
     ``mode`` "logistic": the score is z = router.x (float32 sums) and the weight its logistic function.
     ``mode`` "softmax": s = softmax(z) over all experts, the choice goes by s + ``correction`` (float32 [experts],
     no part of the weights) and the weights are the chosen s over their sum (+ 1e-20).  In that mode the experts may
     form ``groups`` equal groups of neighbours, of which only the ``keep`` with the largest best score stay open to
-    the choice; ``renorm`` False leaves the chosen s undivided; ``scale`` multiplies the weights."""
+    the choice; ``renorm`` False leaves the chosen s undivided; ``scale`` multiplies the weights.
+    ``mode`` "softmax_chosen": the choice goes by z and the weights are the softmax over the chosen z alone.
+    ``bias`` (float32 [experts]) is added to z in every mode."""
     assert x.dtype == router.dtype and x.stride(1) == 1 and router.is_contiguous() and router.shape[1] == x.shape[1]
     assert ids.dtype == torch.int32 and weights.dtype == torch.float32 and ids.is_contiguous() and weights.is_contiguous()
     assert ids.shape == (x.shape[0], top) and weights.shape == ids.shape
-    _check_route(mode, correction, router.shape[0])
+    _check_route(mode, correction, router.shape[0], bias)
     opts = _route_opts(mode, router.shape[0], top, groups, keep, renorm, scale)
     f = _fn("grouped", "brolm_route_topk", [c_int, c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
-                                            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
+                                            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
     _check(f(_code(x), _ptr(x), x.stride(0), _ptr(router), x.shape[0], router.shape[0], x.shape[1], top, _ptr(ids),
-             _ptr(weights), ROUTE_MODES[mode], _ptr(correction), *opts, _stream()), "route_topk")
+             _ptr(weights), ROUTE_MODES[mode], _ptr(correction), *opts, _ptr(bias), _stream()), "route_topk")
 
 
 def route_pick(z: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, mode: str = "logistic",
                correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, renorm: bool = True,
-               scale: float = 1.0) -> None:
+               scale: float = 1.0, bias: Optional[torch.Tensor] = None) -> None:
     """The choice of ``route_topk`` from scores z [tokens, experts] float32 that a matrix product left in memory."""
     assert z.dtype == torch.float32 and z.dim() == 2 and z.stride(1) == 1 and z.shape[1] <= 1024
     assert ids.dtype == torch.int32 and weights.dtype == torch.float32 and ids.is_contiguous() and weights.is_contiguous()
     assert ids.shape == (z.shape[0], top) and weights.shape == ids.shape
-    _check_route(mode, correction, z.shape[1])
+    _check_route(mode, correction, z.shape[1], bias)
     opts = _route_opts(mode, z.shape[1], top, groups, keep, renorm, scale)
     f = _fn("grouped", "brolm_route_pick", [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
-                                            c_int, c_int, c_int, c_float, c_void_p])
+                                            c_int, c_int, c_int, c_float, c_void_p, c_void_p])
     _check(f(_ptr(z), z.stride(0), z.shape[0], z.shape[1], top, _ptr(ids), _ptr(weights), ROUTE_MODES[mode],
-             _ptr(correction), *opts, _stream()), "route_pick")
+             _ptr(correction), *opts, _ptr(bias), _stream()), "route_pick")
 
 
 GROUP_ROWS = 64          # rows of a tile of the grouped product
@@ -549,7 +553,7 @@ def qkv_finish(proj: torch.Tensor, bias: Optional[torch.Tensor], n_q: int, n_kv:
     every q and k head rotated with ``cos_sin`` [positions, rotary_dim / 2, 2], pairs (i, i + rotary_dim / 2)
     ("half") or (2i, 2i + 1) ("interleaved"); v <- (1 - mix) v + mix v_first with ``mix`` a float32 scalar on
     the device and ``v_first`` float32 (tokens, n_kv * v_dim); ``v_keep`` (float32, contiguous) takes this layer's
-    own values as they are before the mixing; the result in ``out``'s element type into ``out`` and the cache."""
+    own values as they are before the mixing; ``n_kv`` may be 0 (queries alone); the result in ``out``'s element type into ``out`` and the cache."""
     cols = (n_q + n_kv) * head_dim + n_kv * v_dim
     parts, part_stride = (proj.shape[0], proj.stride(0)) if proj.dim() == 3 else (1, 0)
     assert proj.shape[-1] == cols and proj.stride(-1) == 1 and out.stride(1) == 1 and out.shape == (proj.shape[-2], cols)
@@ -700,6 +704,26 @@ def norm_sigmoid_gate(y: torch.Tensor, z: torch.Tensor, gain: Optional[torch.Ten
              eps, cols, _ptr(out), _code(out), out.stride(0), tokens, _stream()), "norm_sigmoid_gate")
 
 
+HEAD_GATES = {"silu": 0, "sigmoid": 1}
+
+
+def head_norm_gate(y: torch.Tensor, z: torch.Tensor, gain: Optional[torch.Tensor], eps: float, heads: int, gate: str,
+                   out: torch.Tensor) -> None:
+    """out = n(y) * gate(z) row by row, n dividing every one of ``heads`` equal parts of y by its own
+    sqrt(mean(part^2) + eps), times ``gain`` (float32, one number a column) when given; ``gate`` "silu" or "sigmoid".
+    y, z float32 (tokens, cols), possibly strided views."""
+    tokens, cols = y.shape
+    assert y.dtype == torch.float32 and z.dtype == torch.float32 and z.shape == y.shape and out.shape == y.shape
+    assert y.stride(1) == 1 and z.stride(1) == 1 and out.stride(1) == 1 and heads > 0 and cols % heads == 0
+    assert gain is None or (gain.dtype == torch.float32 and gain.is_contiguous() and gain.numel() == cols)
+    if gate not in HEAD_GATES:
+        raise KernelError(f"head_norm_gate: unknown gate '{gate}' (known: {sorted(HEAD_GATES)})")
+    f = _fn("rowwise", "brolm_head_norm_gate", [c_void_p, c_long, c_void_p, c_long, c_void_p, c_float, c_int, c_int, c_int,
+                                                c_void_p, c_int, c_long, c_int, c_void_p])
+    _check(f(_ptr(y), y.stride(0), _ptr(z), z.stride(0), _ptr(gain), eps, heads, cols // heads, HEAD_GATES[gate], _ptr(out),
+             _code(out), out.stride(0), tokens, _stream()), "head_norm_gate")
+
+
 # --- mixers with a state (csrc/recurrent.cu) --------------------------------
 CONV_ACTS = {"none": 0, "silu": 1}
 
@@ -830,15 +854,29 @@ def decay_state_size(heads: int, dim: int, v_dim: int) -> int:
     return heads * v_dim * ((dim + 3) // 4 * 4)
 
 
+def _head_table(cos_sin: Optional[torch.Tensor], dim: int) -> int:
+    """How many entries of a head the table rotates (0 without one)."""
+    if cos_sin is None:
+        return 0
+    assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.dim() == 3 and cos_sin.shape[2] == 2
+    assert 0 < 2 * cos_sin.shape[1] <= dim
+    return 2 * cos_sin.shape[1]
+
+
 def decay_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, dim: int, v_dim: int, activation: str,
                decay_m1: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
-               out: torch.Tensor, batch: int, max_q_len: int = 0) -> None:
+               out: torch.Tensor, batch: int, max_q_len: int = 0, cos_sin: Optional[torch.Tensor] = None,
+               k_scale: float = 1.0) -> None:
     """Linear attention with a fixed decay per head over the packed tokens: S <- decay_h S + k v^T, out = S^T q.
     q, k (``dim`` per head) and v (``v_dim`` per head) are columns of ``qkv`` (tokens, cols) from ``q_off``, ``k_off``,
     ``v_off`` on, head by head; ``activation`` ("none", "silu") is applied to them as they are read.  ``decay_m1``
     float32 [heads] holds decay - 1.  S is the first ``decay_state_size`` floats of ``state[slot]``.  ``out`` float32
     (tokens, heads * v_dim).  ``max_q_len`` 1 says that every sequence brings one token (the launch then takes part
-    in programmatic launch); 0: unknown."""
+    in programmatic launch); 0: unknown.  ``cos_sin`` (float32 [positions, r / 2, 2]) rotates the first r entries of
+    every q and k head by the token's position (pairs (i, i + r / 2)) and ``k_scale`` multiplies k, both in float as
+    the rows are read, after the activation (float32 rows only)."""
+    rot = _head_table(cos_sin, dim)
+    assert (rot == 0 and k_scale == 1.0) or qkv.dtype == torch.float32
     assert qkv.stride(1) == 1 and out.dtype == torch.float32 and out.stride(1) == 1 and out.shape == (qkv.shape[0], heads * v_dim)
     assert decay_m1.dtype == torch.float32 and decay_m1.is_contiguous() and decay_m1.numel() == heads
     assert max(q_off, k_off) + heads * dim <= qkv.shape[1] and v_off + heads * v_dim <= qkv.shape[1]
@@ -847,10 +885,23 @@ def decay_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
         raise KernelError(f"decay_scan: unknown activation '{activation}'")
     f = _fn("linear_attn", "brolm_decay_scan", [c_void_p, c_int, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_long,
-                                                c_int, c_int, c_void_p])
+                                                c_int, c_int, c_void_p, c_int, c_float, c_void_p])
     _check(f(_ptr(qkv), _code(qkv), qkv.stride(0), q_off, k_off, v_off, heads, dim, v_dim, SCAN_ACTS[activation],
-             _ptr(decay_m1), *_seq(cu_q, kv_len, slots, state), _ptr(out), out.stride(0), batch, int(max_q_len), _stream()),
-           "decay_scan")
+             _ptr(decay_m1), *_seq(cu_q, kv_len, slots, state), _ptr(out), out.stride(0), batch, int(max_q_len),
+             _ptr(cos_sin), rot, float(k_scale), _stream()), "decay_scan")
+
+
+def rotate_heads(rows: torch.Tensor, q_off: int, k_off: int, heads: int, dim: int, positions: torch.Tensor,
+                 cos_sin: Optional[torch.Tensor], k_scale: float = 1.0) -> None:
+    """In place on float32 ``rows`` (tokens, cols): the rotation and the scale of k that ``decay_scan`` applies itself to
+    a step of single tokens, for the heads of q at column ``q_off`` and of k at ``k_off``."""
+    assert rows.dtype == torch.float32 and rows.stride(1) == 1 and positions.dtype == torch.int32
+    assert positions.numel() == rows.shape[0] and max(q_off, k_off) + heads * dim <= rows.shape[1]
+    rot = _head_table(cos_sin, dim)
+    f = _fn("linear_attn", "brolm_rotate_heads", [c_void_p, c_long, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                                                  c_float, c_int, c_void_p])
+    _check(f(_ptr(rows), rows.stride(0), q_off, k_off, heads, dim, _ptr(positions), _ptr(cos_sin), rot, float(k_scale),
+             rows.shape[0], _stream()), "rotate_heads")
 
 
 def linear_f32(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> None:
@@ -1525,5 +1576,5 @@ __all__ = ["KernelBuildError", "KernelError", "build_all", "launch_count", "devi
            "experts_linear", "rmsnorm", "residual_rmsnorm",
            "rope_kv_write", "rope_kv_write_parts", "gated_act", "softcap", "linear_f32", "skinny_gemm", "skinny_qkv_rope", "skinny_ok", "skinny_parts", "skinny_rope_tiles", "gemm_tc", "gemm_tc2", "gemm_tc2_status", "gemm_tc_ok", "gemm_tc_status", "gemm_stream", "gemm_stream_ok", "gemm_stream_parts", "stream_rows",
            "gemm_stream_status", "attention_simt", "attention_prefill_mma", "attention_prefill_tc", "attention_prefill_tc_ok", "attention_prefill_tc_split", "attention_tc_status", "attention_decode_mma",
-           "decode_splits", "argmax", "sample", "cast", "bias_act", "scaled_sum", "qkv_norm_write", "gate_group_norm",
+           "decode_splits", "argmax", "sample", "cast", "bias_act", "scaled_sum", "qkv_norm_write", "gate_group_norm", "head_norm_gate", "rotate_heads",
            "experts_combine", "causal_conv", "conv_tail", "gated_scan", "ssm_scan", "block_matvec_f32", "block_matvec_ok", "split_halves"]

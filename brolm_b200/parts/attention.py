@@ -21,7 +21,7 @@ A third set of options works one head at a time between the projection and
 the attention (``headwise``; the notation: H query heads, G key/value heads,
 head h reads kv head h // (H / G)):
 
-* ``bias``: q, k, v and the output projection have a bias each;
+* ``bias``: q, k, v and the output projection have a bias each; "qkv": only q, k and v have one;
 * ``taps`` = K > 0: a causal convolution per channel over time on the projected
   q, k and v (``y_t = sum_j w[:, j] u_(t - K + 1 + j)``, zeros before the
   sequence's start), whose last K - 1 inputs are kept per sequence in a state
@@ -32,7 +32,8 @@ head h reads kv head h // (H / G)):
   all key heads (``k_norm``);
 * ``sink``: a learned number per query head (tensor ``sink``) whose exponential
   joins the softmax's denominator: it has no key and no value, and is neither
-  scaled nor capped;
+  scaled nor capped; "zero": no tensor, every head's number is 0, so that the
+  weights are exp(s_j) / (1 + sum exp(s_j));
 * ``distance_rows`` = B > 0 with ``distance_far`` = D: a learned bias by distance
   (tensor ``rel``, B rows of one number per query head) is added to the score
   after the scale and the cap; key j at distance n = p - j reads row n for
@@ -56,7 +57,16 @@ head h reads kv head h // (H / G)):
 * ``v_mix``: "source" leaves the layer's values of the step's tokens (float,
   before rounding) under ``v_mix_key`` for later layers of the same pass;
   "mixed" makes v <- (1 - lambda) v + lambda v_source with a learned scalar
-  lambda, and that is what the cache keeps.  Both hold a tensor ``vmix``.
+  lambda, and that is what the cache keeps.  Both hold a tensor ``vmix``;
+* keys and values shared between layers: a layer with ``lends_kv`` leaves the
+  keys (normed, rotated) and values of a prompt step's tokens, in the step's
+  element type, for the layers that read them; a layer with ``borrows_kv`` has
+  no key and value projections and attends to the keys and values of the
+  schedule entry whose cache it is given (``LayerCall.cache_of``): a prompt to
+  the packed rows that entry's layer left in this step (a window's ring no
+  longer holds all of them), a decode step to that entry's pages.  Queries,
+  scale, cap, mask and sink are its own; the entry's cache is wide enough for
+  both masks (``cache.shared_spec``).
 """
 from __future__ import annotations
 
@@ -94,15 +104,16 @@ class Attention(Part):
 
     def __init__(self, hidden: int, n_q: int, n_kv: int, head_dim: int, scale: float, softcap: float = 0.0,
                  window: Optional[int] = None, position: Optional[Part] = None, v_dim: Optional[int] = None,
-                 qk_norm: str = "none", eps: float = 0.0, chunk: Optional[int] = None, bias: bool = False, taps: int = 0,
+                 qk_norm: str = "none", eps: float = 0.0, chunk: Optional[int] = None, bias=False, taps: int = 0,
                  slope_power: float = 0.0, keep_first: int = 0, talk: bool = False, gate: bool = False,
-                 v_mix: Optional[str] = None, v_mix_key: str = "v_first", qk_gain: bool = False, sink: bool = False,
-                 distance_rows: int = 0, distance_far: float = 0.0, distance_rows_free: bool = False):
+                 v_mix: Optional[str] = None, v_mix_key: str = "v_first", qk_gain: bool = False, sink=False,
+                 distance_rows: int = 0, distance_far: float = 0.0, distance_rows_free: bool = False,
+                 lends_kv: bool = False, borrows_kv: bool = False):
         if n_q % n_kv:
             raise ValueError("attention: the number of query heads must be a multiple of the kv heads")
         rotation = getattr(position, "pairing", "half")
         self.headwise = bool(bias or taps or qk_norm == "head" or slope_power or keep_first or talk or gate or v_mix
-                             or sink or distance_rows
+                             or sink or distance_rows or lends_kv or borrows_kv
                              or (position is not None and ((v_dim and v_dim != head_dim) or rotation != "half")))
         plain = not (v_dim and v_dim != head_dim) and qk_norm == "none" and not chunk and not self.headwise
         if plain and head_dim % 16:
@@ -127,6 +138,13 @@ class Attention(Part):
             raise ValueError("attention: the distance bias needs at least two rows and distance_far beyond half of them")
         if (sink or distance_rows) and talk:
             raise ValueError("attention: a sink or a distance bias together with mixed heads' weights is not built")
+        if bias not in (False, True, None, "qkv"):
+            raise ValueError(f"attention: unknown bias '{bias}' (True, 'qkv')")
+        if sink not in (False, True, None, "zero"):
+            raise ValueError(f"attention: unknown sink '{sink}' (True, 'zero')")
+        if borrows_kv and (taps or v_mix or lends_kv):
+            raise ValueError("attention: a layer that reads another layer's keys and values has no convolution and no "
+                             "value mixing of its own, and lends nothing on")
         if keep_first and chunk:
             raise ValueError("attention: kept first keys together with a chunked mask are not built")
         self.hidden, self.n_q, self.n_kv, self.head_dim = hidden, n_q, n_kv, head_dim
@@ -140,10 +158,12 @@ class Attention(Part):
         # the options of the second paragraph above: their own row-wise kernel and the exact attention
         self.bias, self.taps, self.slope_power, self.keep_first = bool(bias), int(taps), float(slope_power), int(keep_first)
         self.talk, self.gate, self.v_mix, self.v_mix_key = bool(talk), bool(gate), v_mix, v_mix_key
-        self.qk_gain, self.has_sink = bool(qk_gain), bool(sink)
+        self.qk_gain, self.has_sink, self.null_sink = bool(qk_gain), bool(sink), sink == "zero"
+        self.has_o_bias = bool(bias) and bias != "qkv"
+        self.lends_kv, self.borrows_kv = bool(lends_kv), bool(borrows_kv)
         self.distance_rows, self.distance_far = int(distance_rows), float(distance_far)
         self.distance_rows_free = bool(distance_rows_free)
-        self.cols = self.q_dim + self.kv_dim + self.v_cols
+        self.cols = self.q_dim if self.borrows_kv else self.q_dim + self.kv_dim + self.v_cols
         self.slopes = None
         self.rowwise = (self.v_dim != head_dim or qk_norm != "none" or self.chunk is not None) and not self.headwise
         if self.headwise and (self.v_dim > 512 or n_q > 128):
@@ -157,20 +177,26 @@ class Attention(Part):
     def param_specs(self):
         specs = {"q": ParamSpec((self.q_dim, self.hidden)), "k": ParamSpec((self.kv_dim, self.hidden)),
                  "v": ParamSpec((self.v_cols, self.hidden)), "o": ParamSpec((self.hidden, self.n_q * self.v_dim))}
+        if self.borrows_kv:
+            del specs["k"], specs["v"]
         if self.qk_norm == "whole":
             specs["q_norm"] = ParamSpec((self.q_dim,), "vector")
             specs["k_norm"] = ParamSpec((self.kv_dim,), "vector")
         if self.qk_gain:
             specs["q_norm"] = ParamSpec((self.head_dim,), "vector")
-            specs["k_norm"] = ParamSpec((self.head_dim,), "vector")
-        if self.has_sink:
+            if not self.borrows_kv:
+                specs["k_norm"] = ParamSpec((self.head_dim,), "vector")
+        if self.has_sink and not self.null_sink:
             specs["sink"] = ParamSpec((self.n_q,), "vector")
         if self.distance_rows:
             specs["rel"] = ParamSpec((-self.distance_rows if self.distance_rows_free else self.distance_rows, self.n_q),
                                      "vector")
         if self.bias:
-            specs.update(q_bias=ParamSpec((self.q_dim,), "vector"), k_bias=ParamSpec((self.kv_dim,), "vector"),
-                         v_bias=ParamSpec((self.v_cols,), "vector"), o_bias=ParamSpec((self.hidden,), "vector"))
+            specs["q_bias"] = ParamSpec((self.q_dim,), "vector")
+            if not self.borrows_kv:
+                specs.update(k_bias=ParamSpec((self.kv_dim,), "vector"), v_bias=ParamSpec((self.v_cols,), "vector"))
+        if self.has_o_bias:
+            specs["o_bias"] = ParamSpec((self.hidden,), "vector")
         if self.taps:
             specs.update(q_conv=ParamSpec((self.q_dim, self.taps), "vector"), k_conv=ParamSpec((self.kv_dim, self.taps), "vector"),
                          v_conv=ParamSpec((self.v_cols, self.taps), "vector"))
@@ -184,23 +210,29 @@ class Attention(Part):
 
     def bind(self, params):
         # one projection for q, k and v: rows [Wq; Wk; Wv]
-        kinds = {params[n].dtype for n in ("q", "k", "v")}
+        own = ("q",) if self.borrows_kv else ("q", "k", "v")
+        kinds = {params[n].dtype for n in own}
         dt = torch.float32 if (len(kinds) > 1 or torch.float32 in kinds) else next(iter(kinds))
-        rows = [params["q"].to(dt), params["k"].to(dt), params["v"].to(dt)]
+        rows = [params[n].to(dt) for n in own]
         if self.gate:
             rows.append(params["gate"].to(dt))               # the gates' logits are columns of the same product
         self.w_qkv = torch.cat(rows, dim=0).contiguous()
         self.w_o = params["o"]
         f32 = lambda *names: torch.cat([params[n].float() for n in names], dim=0).contiguous()
-        self.in_bias = f32("q_bias", "k_bias", "v_bias") if self.bias else None
-        self.o_bias = params["o_bias"].float().contiguous() if self.bias else None
+        self.in_bias = f32(*[n + "_bias" for n in own]) if self.bias else None
+        self.o_bias = params["o_bias"].float().contiguous() if self.has_o_bias else None
         self.conv = f32("q_conv", "k_conv", "v_conv") if self.taps else None
         self.w_talk = params["talk"].float().contiguous() if self.talk else None
         self.lam = params["vmix"].float().reshape(1).contiguous() if self.v_mix == "mixed" else None
         self.q_gain = self.k_gain = None
         if self.qk_gain:
-            self.q_gain, self.k_gain = params["q_norm"].float().contiguous(), params["k_norm"].float().contiguous()
-        self.sink = params["sink"].float().contiguous() if self.has_sink else None
+            self.q_gain = params["q_norm"].float().contiguous()
+            self.k_gain = params["k_norm"].float().contiguous() if not self.borrows_kv else None
+        self.sink = None
+        if self.null_sink:
+            self.sink = torch.zeros(self.n_q, dtype=torch.float32, device=self.w_o.device)
+        elif self.has_sink:
+            self.sink = params["sink"].float().contiguous()
         self.dist_bias = None
         if self.distance_rows:
             # laid out by distance: [head][n] for n up to the first distance that reads the last row (all further do)
@@ -316,8 +348,9 @@ class Attention(Part):
 
     def _forward_headwise(self, x, ctx, entry, writes_cache):
         """The path of a layer with one of the head-wise options of the module's third paragraph."""
-        if not writes_cache:
-            raise NotImplementedError("a layer of this kind cannot run on another layer's cache")
+        if writes_cache == self.borrows_kv:
+            raise NotImplementedError("a layer with keys and values of its own cannot run on another layer's cache, nor one "
+                                      "without them on a cache of its own")
         kv_entry, conv_entry = (entry.parts[0], entry.parts[1]) if self.taps else (entry, None)
         k_pages, v_pages, table, ring, page = ctx.kv(kv_entry)
         T, cols, dev = x.shape[0], self.cols, x.device
@@ -338,14 +371,27 @@ class Attention(Part):
             mix, v_first = self.lam, ctx.carry[self.v_mix_key]
         qkv = torch.empty((T, cols), dtype=ctx.dtype, device=dev)
         pos = self.position
-        kernels.qkv_finish(rows, bias, self.n_q, self.n_kv, self.head_dim, self.v_dim, ctx.positions, qkv,
+        kept = dict(k_pages=k_pages, v_pages=v_pages, cache_rows=ctx.cache_rows[kv_entry.group_id], page_size=page) \
+            if writes_cache else {}
+        kernels.qkv_finish(rows, bias, self.n_q, 0 if self.borrows_kv else self.n_kv, self.head_dim, self.v_dim,
+                           ctx.positions, qkv,
                            head_norm=self.qk_norm == "head", eps=self.eps,
                            cos_sin=pos.table if pos is not None else None,
                            rotary_dim=pos.rotary_dim if pos is not None else 0,
                            pairing=pos.pairing if pos is not None else "half", mix=mix, v_first=v_first, v_keep=v_keep,
-                           q_gain=self.q_gain, k_gain=self.k_gain, k_pages=k_pages, v_pages=v_pages, cache_rows=ctx.cache_rows[kv_entry.group_id], page_size=page)
+                           q_gain=self.q_gain, k_gain=self.k_gain, **kept)
         q = qkv[:, :self.q_dim]
-        k, v = qkv[:, self.q_dim:self.q_dim + self.kv_dim], qkv[:, self.q_dim + self.kv_dim:]
+        shared = ("kv", kv_entry.group_id, kv_entry.index)
+        if not self.borrows_kv:
+            k, v = qkv[:, self.q_dim:self.q_dim + self.kv_dim], qkv[:, self.q_dim + self.kv_dim:]
+            if self.lends_kv and ctx.mode == "prefill":
+                ctx.carry[shared] = (k, v)
+        elif ctx.mode == "prefill":
+            if shared not in ctx.carry:
+                raise RuntimeError("attention: the layer whose keys and values this one reads left none in this pass")
+            k, v = ctx.carry[shared]
+        else:
+            k = v = None                      # a decode step reads the pages
         group = self.n_q // self.n_kv
         common = dict(n_kv=self.n_kv, group=group, head_dim=self.head_dim, scale=self.scale, cap=self.softcap,
                       window=self.window or 0, batch=ctx.batch, max_q_len=ctx.max_q_len)

@@ -38,7 +38,11 @@ class RoutedExperts(Part):
     * ``groups`` = (count, keep) with the softmax router: the experts form ``count`` equal groups of neighbours, a
       group's score is its largest s (+ correction), and only experts of the ``keep`` best groups can be chosen;
     * ``renorm=False`` with the softmax router: the weights are the chosen s themselves, not divided by their sum;
-    * ``weight_scale``: a constant that multiplies the weights.
+    * ``weight_scale``: a constant that multiplies the weights;
+    * ``router="softmax_chosen"``: the ``top`` largest z are chosen and the weights are the softmax over those alone;
+    * ``router_bias``: a learned number per expert is added to z (tensor ``router_bias``); it is part of the score;
+    * ``activation="clamped_gate"`` with ``gated`` and ``limit`` > 0: g = min(gate, limit), u = clamp(up, -limit,
+      limit), the expert is W_down (g sigmoid(1.702 g) (u + 1)).
 
     The result of that form is one float32 (tokens, hidden) array: weights, identity experts and the shared
     expert are folded in by one row-wise kernel.
@@ -50,7 +54,7 @@ class RoutedExperts(Part):
     def __init__(self, hidden: int, inter: int, experts: int, top: int, activation: str = "relu2",
                  scale_input: bool = True, router: str = "logistic", correction: bool = False, gated: bool = False,
                  identity: int = 0, shared: Optional[Part] = None, shared_gate: bool = False, groups=None,
-                 renorm: bool = True, weight_scale: float = 1.0):
+                 renorm: bool = True, weight_scale: float = 1.0, router_bias: bool = False, limit: float = 0.0):
         count, keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
         if (count, keep) != (1, 1) or not renorm or float(weight_scale) != 1.0:
             if router != "softmax":
@@ -63,14 +67,17 @@ class RoutedExperts(Part):
         if shared_gate and shared is None:
             raise ValueError("routed experts: a gate of the shared expert needs a shared expert")
         self.groups, self.keep, self.renorm, self.weight_scale = count, keep, bool(renorm), float(weight_scale)
-        self.has_shared_gate = bool(shared_gate)
+        if activation == "clamped_gate" and not limit > 0:
+            raise ValueError("routed experts: the clamped gate needs a positive limit")
+        self.has_shared_gate, self.has_router_bias, self.limit = bool(shared_gate), bool(router_bias), float(limit)
         if experts < 0 or identity < 0 or not 1 <= top <= experts + identity:
             raise ValueError("routed experts: 1 <= top <= experts + identity")
         if router not in kernels.ROUTE_MODES:
             raise ValueError(f"routed experts: unknown router '{router}'")
         if correction and router != "softmax":
             raise ValueError("routed experts: a correction of the choice goes with the softmax router")
-        self.weighted = bool(router != "logistic" or not scale_input or gated or identity or shared is not None)
+        self.weighted = bool(router != "logistic" or not scale_input or gated or identity or shared is not None
+                             or router_bias)
         self.route_opts = dict(groups=count, keep=keep, renorm=bool(renorm), scale=float(weight_scale)) \
             if router == "softmax" else {}
         if self.weighted:
@@ -94,6 +101,8 @@ class RoutedExperts(Part):
         specs = {"router": ParamSpec((self.experts + self.identity, self.hidden))}
         if self.has_correction:
             specs["correction"] = ParamSpec((self.experts + self.identity,), "vector")
+        if self.has_router_bias:
+            specs["router_bias"] = ParamSpec((self.experts + self.identity,), "vector")
         if self.has_shared_gate:
             specs["shared_gate"] = ParamSpec((1, self.hidden))
         for e in range(self.experts):
@@ -110,6 +119,7 @@ class RoutedExperts(Part):
         if len(kinds) > 1:
             raise TypeError("routed experts: the experts' matrices and the router must have one element type")
         self.correction = params["correction"].float().contiguous() if self.has_correction else None
+        self.router_bias = params["router_bias"].float().contiguous() if self.has_router_bias else None
         self.w_shared_gate = params["shared_gate"].to(self.router.dtype).reshape(-1).contiguous() \
             if self.has_shared_gate else None
         if self.experts:
@@ -127,9 +137,10 @@ class RoutedExperts(Part):
             # a prompt: the scores as one matrix product (bfloat16 products are exact in float, the sums are
             # float), then the choice; the router kernel's float multiply-adds are what bounds it from here on
             kernels.route_pick(linear(x, self.router, out_dtype=torch.float32), self.top, ids, gates, self.route_mode,
-                               self.correction, **self.route_opts)
+                               self.correction, bias=self.router_bias, **self.route_opts)
         else:
-            kernels.route_topk(x, self.router, self.top, ids, gates, self.route_mode, self.correction, **self.route_opts)
+            kernels.route_topk(x, self.router, self.top, ids, gates, self.route_mode, self.correction, bias=self.router_bias,
+                               **self.route_opts)
 
     def _forward_weighted(self, x: torch.Tensor, ctx) -> torch.Tensor:
         """x (tokens, hidden) -> (tokens, hidden) float32: the weighted sum of the chosen experts' results,
@@ -159,7 +170,7 @@ class RoutedExperts(Part):
                 kernels.experts_linear(x, self.w_up, u, perm, offsets, tiles, self.top, T, activation=act)
             if self.gated:
                 a = torch.empty((pairs, self.inter), dtype=x.dtype, device=dev)
-                kernels.gated_act(u, a, self.activation)
+                kernels.gated_act(u, a, self.activation, self.limit)
                 u = a
             y = torch.empty((self.top, T, self.hidden), dtype=torch.float32, device=dev)
             if tc:

@@ -18,18 +18,27 @@ class RMSNorm(Part):
 
     ``groups`` > 1: the row is cut into that many equal consecutive parts and every part is divided by its own
     root mean square; the gain still spans the whole row.
+
+    ``scalar``: the gain is one number for the whole row (a tensor of shape ()); it is spread over a row when the
+    tensors are bound, so every kernel that takes a gain row takes it.
     """
 
     kind = "norm"
     graph_safe = True
 
-    def __init__(self, size: int, eps: float, offset: float = 0.0, groups: int = 1):
+    def __init__(self, size: int, eps: float, offset: float = 0.0, groups: int = 1, scalar: bool = False):
         if groups < 1 or size % groups:
             raise ValueError(f"norm: {groups} groups do not divide a row of {size}")
         self.size, self.eps, self.offset, self.groups = size, float(eps), float(offset), int(groups)
+        self.scalar = bool(scalar)
 
     def param_specs(self):
-        return {"weight": ParamSpec((self.size,), "vector")}
+        return {"weight": ParamSpec(() if self.scalar else (self.size,), "vector")}
+
+    def bind(self, params):
+        if self.scalar:
+            params = {"weight": params["weight"].reshape(1).expand(self.size).contiguous()}
+        super().bind(params)
 
     @property
     def weight(self) -> torch.Tensor:

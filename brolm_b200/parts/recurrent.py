@@ -8,6 +8,8 @@ a prompt and a decode step, and nothing is read back to the host.
 """
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import kernels
@@ -188,13 +190,18 @@ class DecayLinearAttention(Part):
     head; per head S <- decay_h S + k v^T and o = S^T q, with no other scale.  The heads' results together pass an
     RMS norm over the whole row with a gain (``norm``), are multiplied by sigmoid(W_g x) (``gate``) and go through
     W_o.  ``decay``: one number per head.  The projection's sums, the activation, S and the norm are float32 in
-    every mode; S is a state row per sequence, zero at the sequence's start."""
+    every mode; S is a state row per sequence, zero at the sequence's start.
+
+    Options: ``position`` rotates the first entries of every q and k head by the token's position, ``k_scale``
+    multiplies k after that (retention: Sun et al., "Retentive Network: A Successor to Transformer for Large Language
+    Models"); both act on the projection's float sums.  ``norm="head"``: every head's result is divided by its own
+    root mean square, without a gain.  ``gate="silu"``: the results are multiplied by silu(W_g x)."""
 
     kind = "mixer"
     graph_safe = True
 
     def __init__(self, hidden: int, heads: int, dim: int, v_dim: int, decay, eps: float, activation: str = "silu",
-                 norm: bool = True, gate: bool = True):
+                 norm=True, gate=True, position: Optional[Part] = None, k_scale: float = 1.0):
         decay = [float(d) for d in decay]
         if len(decay) != heads:
             raise ValueError(f"decay attention: {len(decay)} decays for {heads} heads")
@@ -204,8 +211,18 @@ class DecayLinearAttention(Part):
             raise ValueError(f"decay attention: unknown activation '{activation}'")
         if dim > 512:
             raise ValueError("decay attention: more than 512 query/key entries per head are beyond the kernel")
+        if norm not in (True, False, "head") or gate not in (True, False, "sigmoid", "silu"):
+            raise ValueError(f"decay attention: unknown norm '{norm}' or gate '{gate}'")
+        if norm == "head" and not gate:
+            raise ValueError("decay attention: a norm per head without a gate is not built")
+        if norm != "head" and gate == "silu":
+            raise ValueError("decay attention: a silu gate goes with the norm per head")
+        if position is not None and (position.pairing != "half" or position.rotary_dim > dim):
+            raise ValueError("decay attention: the rotation pairs entries i and i + r/2 of a head's first r")
+        self.position, self.k_scale = position, float(k_scale)
+        self.head_norm, self.gate_act = norm == "head", "silu" if gate == "silu" else "sigmoid"
         self.hidden, self.heads, self.dim, self.v_dim, self.decay = hidden, heads, dim, v_dim, decay
-        self.eps, self.activation, self.has_norm, self.has_gate = float(eps), activation, bool(norm), bool(gate)
+        self.eps, self.activation, self.has_norm, self.has_gate = float(eps), activation, norm is True, bool(gate)
         self.qk_cols, self.v_cols = heads * dim, heads * v_dim
 
     def param_specs(self):
@@ -233,6 +250,10 @@ class DecayLinearAttention(Part):
     def cache_spec(self):
         return StateSpec((kernels.decay_state_size(self.heads, self.dim, self.v_dim),), torch.float32)
 
+    def prepare(self, max_positions, device):
+        if self.position is not None:
+            self.position.prepare(max_positions, device)
+
     def forward(self, x: torch.Tensor, ctx, entry, writes_cache: bool = True) -> torch.Tensor:
         """x (tokens, hidden) -> (tokens, hidden) float32, or partial sums [parts, tokens, hidden]."""
         if not writes_cache:
@@ -247,9 +268,18 @@ class DecayLinearAttention(Part):
             qkv = proj[:, :2 * self.qk_cols + self.v_cols]
             kernels.bias_act(qkv, None, act, qkv)
             act = "none"
+        table, k_scale = self.position.table if self.position is not None else None, self.k_scale
+        if (table is not None or k_scale != 1.0) and ctx.max_q_len > 1:
+            # the same for the rotation and k's scale (after the activation, as in the scan)
+            kernels.rotate_heads(proj, 0, self.qk_cols, self.heads, self.dim, ctx.positions, table, k_scale)
+            table, k_scale = None, 1.0
         kernels.decay_scan(proj, 0, self.qk_cols, 2 * self.qk_cols, self.heads, self.dim, self.v_dim, act,
-                           self.decay_m1, ctx.cu_q, ctx.kv_len, ctx.slots_dev, ctx.state(entry), y, ctx.batch, ctx.max_q_len)
-        if self.has_norm or self.has_gate:
+                           self.decay_m1, ctx.cu_q, ctx.kv_len, ctx.slots_dev, ctx.state(entry), y, ctx.batch, ctx.max_q_len,
+                           cos_sin=table, k_scale=k_scale)
+        if self.head_norm:
+            out = torch.empty((T, self.v_cols), dtype=ctx.dtype, device=x.device)
+            kernels.head_norm_gate(y, proj[:, 2 * self.qk_cols + self.v_cols:], None, self.eps, self.heads, self.gate_act, out)
+        elif self.has_norm or self.has_gate:
             out = torch.empty((T, self.v_cols), dtype=ctx.dtype, device=x.device)
             if self.has_gate:
                 kernels.norm_sigmoid_gate(y, proj[:, 2 * self.qk_cols + self.v_cols:], self.gain, self.eps, out)

@@ -21,7 +21,8 @@ KINDS = ("mixer", "feedforward", "norm", "position", "block", "stream")
 @dataclasses.dataclass(frozen=True)
 class ParamSpec:
     """One tensor a part needs.  ``role``: ``matrix`` (a projection, (out, in)),
-    ``vector`` (a gain or bias), ``table`` (looked up by index), ``int`` (an
+    ``vector`` (a gain or bias), ``gain`` (a vector that scales by itself: made at random it lies around 1),
+    ``table`` (looked up by index), ``int`` (an
     integer table, kept as int32).  A negative entry of ``shape`` leaves that size to the checkpoint's tensor; its
     magnitude is the size a tensor made at random gets."""
     shape: tuple

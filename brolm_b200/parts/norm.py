@@ -33,7 +33,7 @@ class RMSNorm(Part):
         self.scalar = bool(scalar)
 
     def param_specs(self):
-        return {"weight": ParamSpec(() if self.scalar else (self.size,), "vector")}
+        return {"weight": ParamSpec((), "gain") if self.scalar else ParamSpec((self.size,), "vector")}
 
     def bind(self, params):
         if self.scalar:

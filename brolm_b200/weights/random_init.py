@@ -13,7 +13,7 @@ tensors exist or on the order they are made in.
 
 The sum of twelve uniform numbers has mean 6 and variance 1 (Irwin-Hall), so
 value is N(0, std) to the eye, within +-6 std.  Matrices and tables use
-``weight_std``, gain vectors ``norm_std``; the result is rounded once more to
+``weight_std``, gain vectors ``norm_std`` (a gain that scales by itself lies around 1: value + 1); the result is rounded once more to
 the storage type.  wlejon/brolm has no such mode; its tests write a
 uniform(-0.1, 0.1) fixture (tests/test_gemma2.cpp:97-106).
 """
@@ -94,6 +94,9 @@ def random_tensors(expected: dict[str, Expected], seed: int, weight_std: float, 
         shape = tuple(abs(int(n)) for n in e.shape)        # a size left to the tensor: its magnitude when made at random
         if e.role == "int":
             yield name, torch.zeros(shape, dtype=torch.int32, device=device)
+            continue
+        if e.role == "gain":
+            yield name, (random_tensor(seed, name, shape, norm_std, torch.float32, device) + 1.0).to(dtype)
             continue
         yield name, random_tensor(seed, name, shape, norm_std if e.role == "vector" else weight_std, dtype, device)
 

@@ -13,6 +13,12 @@ import torch
 F64 = torch.float64
 
 
+def kept(x):
+    """Every result that a run in a 16-bit element type rounds before the next product passes through here; a test that
+    asks how large an error rounding alone makes puts a rounding in its place (``rounded_forward``)."""
+    return x
+
+
 def unit_rms(x, eps):
     return x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps)
 
@@ -23,7 +29,7 @@ def silu(z):
 
 def scalar_norm(x, gain, eps):
     """The norm of a layer and of the output: one number multiplies every coordinate of the unit row."""
-    return unit_rms(x, eps) * gain
+    return kept(unit_rms(x, eps) * gain)
 
 
 # --- rotation ------------------------------------------------------------------------------------------------------
@@ -89,20 +95,20 @@ def windowed_attention(q, k, v, scale, cap, window, null_sink=True, first=0):
     return torch.stack(heads, dim=1)
 
 
-def attention(n, t, p, m, kept):
-    """``kept``: layer index -> (rotated keys, values) of the attention layers so far that have their own; the layer
-    adds its pair under ``kept["here"]`` unless it reads another layer's."""
+def attention(n, t, p, m, lent):
+    """``lent``: layer index -> (rotated keys, values) of the attention layers so far that have their own; the layer
+    adds its pair under ``lent["here"]`` unless it reads another layer's."""
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     T = n.shape[0]
     q = rotate((n @ t[p + "q"].T + t[p + "q.b"]).view(T, H, d), m["rot"])
     if m.get("kv_from") is not None:
-        k, v = kept[m["kv_from"]]
+        k, v = lent[m["kv_from"]]
     else:
         k = rotate((n @ t[p + "k"].T + t[p + "k.b"]).view(T, G, d), m["rot"])
         v = (n @ t[p + "v"].T + t[p + "v.b"]).view(T, G, dv)
-        kept["here"] = (k, v)
-    o = windowed_attention(q, k, v, m["scale"], m.get("softcap") or 0.0, (m.get("mask") or {}).get("size"))
-    return o.reshape(T, H * dv) @ t[p + "o"].T
+        lent["here"] = (k, v)
+    o = windowed_attention(kept(q), kept(k), kept(v), m["scale"], m.get("softcap") or 0.0, (m.get("mask") or {}).get("size"))
+    return kept(o.reshape(T, H * dv)) @ t[p + "o"].T
 
 
 # --- retention -----------------------------------------------------------------------------------------------------
@@ -127,14 +133,14 @@ def retention(n, t, p, m, eps):
     v = (n @ t[p + "v"].T).view(T, H, dv)
     o, _ = decayed_state(q, k, v, torch.tensor(m["decay"], dtype=F64).to(q.dtype))
     o = unit_rms(o, eps).reshape(T, H * dv)                    # every head by its own root mean square
-    return (o * silu(n @ t[p + "g"].T)) @ t[p + "o"].T
+    return kept(o * silu(n @ t[p + "g"].T)) @ t[p + "o"].T
 
 
 # --- routed experts ------------------------------------------------------------------------------------------------
 def clamped_expert(n, t, p, limit):
-    g = torch.clamp(n @ t[p + "gate"].T, max=limit)
-    u = torch.clamp(n @ t[p + "up"].T, min=-limit, max=limit)
-    return (g * torch.sigmoid(1.702 * g) * (u + 1.0)) @ t[p + "down"].T
+    g = torch.clamp(kept(n @ t[p + "gate"].T), max=limit)
+    u = torch.clamp(kept(n @ t[p + "up"].T), min=-limit, max=limit)
+    return kept(g * torch.sigmoid(1.702 * g) * (u + 1.0)) @ t[p + "down"].T
 
 
 def choose(z, top: int):
@@ -161,14 +167,14 @@ def forward(config: dict, tensors: dict, tokens, streams=None):
     t = {k: (v.to(F64) if v.is_floating_point() else v) for k, v in tensors.items()}
     eps = float(config["norm"]["eps"])
     x = t["embed"][torch.tensor(tokens)] * float(config["embedding"]["scale"])
-    kept = {}
+    lent = {}
     for i, layer in enumerate(config["layers"]):
         p = f"l{i}."
         n = scalar_norm(x, t[p + "norm1"], eps)
         if layer["type"] == "attention":
-            y = attention(n, t, p + "mix.", layer["mixer"], kept)
-            if "here" in kept:
-                kept[i] = kept.pop("here")
+            y = attention(n, t, p + "mix.", layer["mixer"], lent)
+            if "here" in lent:
+                lent[i] = lent.pop("here")
         else:
             y = retention(n, t, p + "mix.", layer["mixer"], eps)
         if layer.get("mlp") is not None:
@@ -177,3 +183,24 @@ def forward(config: dict, tensors: dict, tokens, streams=None):
         if streams is not None:
             streams.append(x.clone())
     return scalar_norm(x, t["final.norm"], eps) @ t["head"].T
+
+
+def rounded_forward(config: dict, tensors: dict, tokens):
+    """``forward`` with every kept result rounded to bfloat16."""
+    global kept
+    exact = kept
+    kept = lambda x: x.to(torch.bfloat16).to(x.dtype)
+    try:
+        return forward(config, tensors, tokens)
+    finally:
+        kept = exact
+
+
+def rounding_errors(config: dict, tensors: dict, requests):
+    """What rounding alone does to the rows of these requests: every row's largest error relative to its request's
+    largest logit, smallest first."""
+    out = []
+    for p in requests:
+        ref = forward(config, tensors, p)
+        out += ((rounded_forward(config, tensors, p) - ref).abs().amax(dim=1) / ref.abs().max()).tolist()
+    return sorted(out)

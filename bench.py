@@ -30,6 +30,10 @@ a distance bias and a sink, gated latent attention, routed experts chosen among 
 the closest design the library has, Neburax (state-space layers, attention beside a recurrence, routed experts with a
 shared expert), built to the same width, heads, experts and layer count.
 
+``--arch relulix [--size s|m]``: the Relulix design (retention; windowed capped attention with a sink, one layer of which
+reads the other's keys and values; routed experts with a clamped gate) beside the closest design the library has,
+Ritirax, with two lightning and two attention layers of the same sizes and experts.
+
 More than one GPU is not what this library does: ``--gpus N`` with N > 1 says
 so and exits with 2.
 """
@@ -673,6 +677,119 @@ def ritirax_main(args, pk) -> int:
     return 0
 
 
+# --arch relulix: two retention layers and two attention layers (the second reads the first one's keys and values), every
+# layer with routed experts; beside Ritirax with two lightning layers and two attention layers of the same width, heads,
+# head sizes and experts (no latent layer, no shared expert, no groups), so that layer stands beside like layer.
+RELULIX_SIZES = {
+    "s": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, rot=64, window=1024, experts=32, top=4, ff=1024, vocab=32768),
+    "m": dict(width=3072, heads=24, kv_heads=4, dim=128, vdim=128, rot=64, window=1024, experts=64, top=6, ff=1024, vocab=65536),
+}
+
+
+def relulix_main(args, pk) -> int:
+    import torch
+
+    import brolm_b200 as bb
+
+    name = args.size if args.size in RELULIX_SIZES else "s"
+    z = RELULIX_SIZES[name]
+    dev = "cuda:0"
+    torch.cuda.set_device(0)
+    W, H, G, d, dv = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"]
+    router = dict(experts=z["experts"], top=z["top"])
+    moe = dict(kind="moe", expert=dict(ff=z["ff"], limit=7.0), router=router)
+    decay = [1.0 - 2.0 ** (-3.0 - 7.0 * h / max(H - 1, 1)) for h in range(H)]
+    ret = dict(heads=H, dim=d, vdim=dv, decay=decay, rot=dict(base=10000.0, dims=d))
+    attn = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=d ** -0.5, softcap=30.0, mask=dict(size=z["window"]),
+                rot=dict(base=10000.0, dims=z["rot"], scaling=dict(factor=8.0, original=1024, fast=32.0, slow=1.0)))
+    layers = [dict(type="retention", mixer=ret, mlp=moe), dict(type="attention", mixer=attn, mlp=moe),
+              dict(type="attention", mixer=dict(attn, kv_from=1), mlp=moe), dict(type="retention", mixer=ret, mlp=moe)]
+    xcfg = bb.RelulixConfig.from_dict(dict(architecture="Relulix", vocab=z["vocab"], width=W, layers=layers,
+                                           norm=dict(eps=1e-5), embedding=dict(scale=W ** 0.5)))
+    cmoe = dict(kind="moe", expert=dict(ff=z["ff"]), router=router)
+    light = dict(heads=H, dim=d, vdim=dv, decay=decay)
+    cattn = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=d ** -0.5, softcap=30.0, bias_max=128, bias_rows=32)
+    clayers = [dict(type="lightning", mixer=light, mlp=cmoe), dict(type="attention", mixer=cattn, mlp=cmoe),
+               dict(type="attention", mixer=cattn, mlp=cmoe), dict(type="lightning", mixer=light, mlp=cmoe)]
+    ccfg = bb.RitiraxConfig.from_dict(dict(architecture="Ritirax", vocab=z["vocab"], width=W, layers=clayers,
+                                           norm=dict(eps=1e-5), embedding=dict(scale=W ** 0.5)))
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    steps, warmup, batch, context, prompt_len = args.steps or 64, max(args.warmup, 3), args.batch or 8, 1280, 2048
+    common = (dev, flush, steps, warmup, batch, context, prompt_len)
+    r, c = measure_design(xcfg, z["vocab"], *common), measure_design(ccfg, z["vocab"], *common)
+    T, ff, top = prompt_len, z["ff"], z["top"]
+    seen = sum(min(t + 1, z["window"]) for t in range(T))                      # visible (query, key) pairs of a prompt
+    keys = T * (T + 1) // 2
+    tf, gb = pk["bf16_burst"] * 1e12, pk["hbm_gbs"] * 1e9
+    active = z["experts"] * (1.0 - (1.0 - top / z["experts"]) ** batch)
+    kv_row, state = G * (d + dv) * 2.0, H * d * dv * 4.0
+    qkv_cols = (H + G) * d + G * dv
+    # (kernel-name fragment, work of all its launches in one pass over the layers, bound)
+    experts = [("grouped_tc_kernel", 4 * 2.0 * T * top * ff * W * 3, "flops"),
+               ("gated_act", 4 * T * top * 3 * ff * 2.0, "bytes"),
+               ("gather_rows", 4 * T * (1 + top) * W * 2.0, "bytes"),
+               ("experts_combine", 4 * T * (top + 1) * W * 4.0, "bytes"),
+               ("route_pick", 4 * T * (z["experts"] + 2 * top) * 4.0, "bytes"),
+               ("residual_rmsnorm", 4 * (3 + 3.5) * T * W * 4.0, "bytes")]
+    scan = ("decay_scan", 2 * T * (H * (2 * d + dv) + H * dv) * 4.0, "bytes")
+    d_experts = [("fast_kernel<64, 64, 4, false>", 4 * active * ff * W * 2.0 * 3, "bytes"),
+                 ("route_kernel", 4 * z["experts"] * W * 2.0, "bytes"),
+                 ("experts_combine", 4 * batch * (top + 1) * W * 4.0, "bytes")]
+    d_scan = ("decay_scan", 2 * batch * state * 2, "bytes")
+    rows = [
+        ("relulix prefill", r["prefill_kernels"], experts + [
+            ("attn_prefill_mma", 2 * 2.0 * H * (d + dv) * seen, "flops"), scan,
+            ("rotate_heads", 2 * T * 2 * H * d * 4.0 * 2, "bytes"),
+            ("head_norm_gate", 2 * T * H * dv * (4 + 4 + 2.0), "bytes"),
+            ("qkv_finish", T * ((qkv_cols + H * d) * 6.0 + kv_row), "bytes"),
+        ]),
+        ("closest prefill", c["prefill_kernels"], experts + [
+            ("attn_prefill_mma", 2 * 2.0 * H * (d + dv) * keys, "flops"), scan,
+            ("bias_act", 2 * T * H * (2 * d + dv) * 4.0 * 2, "bytes"),
+            ("norm_sigmoid_gate", 2 * T * H * dv * (4 + 4 + 2.0), "bytes"),
+            ("qkv_finish", 2 * T * (qkv_cols * 6.0 + kv_row), "bytes"),
+        ]),
+        ("relulix decode", r["decode_kernels"], d_experts + [
+            ("attn_decode_mma", 2 * batch * min(context, z["window"]) * kv_row, "bytes"), d_scan,
+            ("head_norm_gate", 2 * batch * H * dv * 10.0, "bytes"),
+        ]),
+        ("closest decode", c["decode_kernels"], d_experts + [
+            ("attn_decode_mma", 2 * batch * context * kv_row, "bytes"), d_scan,
+            ("norm_sigmoid_gate", 2 * batch * H * dv * 10.0, "bytes"),
+        ]),
+    ]
+    table = []
+    for title, kern, wanted in rows:
+        for frag, work, bound in wanted:
+            us = sum(v["us"] for k, v in kern.items() if frag in k)
+            n = sum(v["n"] for k, v in kern.items() if frag in k)
+            if not n:
+                continue
+            frac = work / (us * 1e-6) / (tf if bound == "flops" else gb)
+            table.append({"step": title, "kernel": frag, "launches": n, "us": round(us, 2),
+                          "bound": "tensor" if bound == "flops" else "hbm", "frac_of_measured_peak": round(frac, 4)})
+    result = {
+        "metric": f"Relulix decode tokens/s (size {name}, batch {batch}, context {context}) beside Ritirax at equal sizes",
+        "value": round(batch * 1000.0 / r["decode_ms"], 1), "unit": "tokens/s", "n_gpus": 1, "steps": steps,
+        "warmup": warmup, "ms_per_step": round(r["decode_ms"], 4), "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",
+        "impl": "brolm_b200", "clocks": r["clocks"], "gpu_launches": r["launches"],
+        "config": {"model": "Relulix", **{k: v for k, v in z.items()}, "layers": len(layers), "global_batch": batch,
+                   "seq_len": context, "closest": {"model": "Ritirax", "layers": [l["type"] for l in clayers]},
+                   "l2": "the prompt is timed after an L2 flush; a decode step reads more than the L2 holds",
+                   "peaks": pk["source"]},
+        "relulix": {"prefill_tok_s": round(T * 1000.0 / r["prefill_ms"], 1), "prefill_ms": round(r["prefill_ms"], 3),
+                    "decode_tok_s": round(batch * 1000.0 / r["decode_ms"], 1), "decode_ms": round(r["decode_ms"], 4)},
+        "closest": {"prefill_tok_s": round(T * 1000.0 / c["prefill_ms"], 1), "prefill_ms": round(c["prefill_ms"], 3),
+                    "decode_tok_s": round(batch * 1000.0 / c["decode_ms"], 1), "decode_ms": round(c["decode_ms"], 4)},
+        "kernels": table,
+        "by_kernel_us": {"relulix_prefill": _top(r["prefill_kernels"], 28), "closest_prefill": _top(c["prefill_kernels"], 28),
+                         "relulix_decode": _top(r["decode_kernels"], 28), "closest_decode": _top(c["decode_kernels"], 28)},
+    }
+    print(json.dumps(result))
+    return 0
+
+
 def _by_kernel(events) -> dict:
     """Device records -> {kernel name: {"us": total time, "n": launches}}."""
     out: dict = {}
@@ -691,9 +808,9 @@ def _top(kern: dict, n: int = 14) -> dict:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--arch", default="gemma2", choices=["gemma2", "banevik", "neburax", "kedasun", "ritirax"],
+    ap.add_argument("--arch", default="gemma2", choices=["gemma2", "banevik", "neburax", "kedasun", "ritirax", "relulix"],
                     help="banevik, neburax, kedasun: that design at real layer sizes beside Gemma 2 at equal sizes (--size s|m); "
-                         "ritirax: beside Neburax at equal sizes")
+                         "ritirax: beside Neburax at equal sizes; relulix: beside Ritirax at equal sizes")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=0, help="decode steps in a timed region (default 64; 128 for 9b)")
     ap.add_argument("--warmup", type=int, default=8)
@@ -723,6 +840,8 @@ def main() -> int:
         return kedasun_main(args, peaks())
     if args.arch == "ritirax":
         return ritirax_main(args, peaks())
+    if args.arch == "relulix":
+        return relulix_main(args, peaks())
     if args.size not in SIZES:
         print(f"bench.py: --size {args.size} goes with --arch banevik, neburax or kedasun")
         return 2

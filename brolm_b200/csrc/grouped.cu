@@ -122,6 +122,35 @@ __device__ __forceinline__ void pick_top(float* zr, int E, int top, int t, int l
         return;
     }
     float first = 0.0f, total = 0.0f;                  // ROUTE_CHOSEN: the largest score, the sum of the exponentials
+    if (mode == ROUTE_CHOSEN && top <= 32) {           // lane k keeps choice k: nothing goes through memory between choices
+        float mine = -INFINITY;
+        int mine_at = 0;
+        for (int k = 0; k < top; ++k) {
+            float best = -INFINITY;
+            int at = 0x7fffffff;
+            for (int e = lane; e < E; e += 32) {
+                const float v = zr[e];
+                if (v > best || (v == best && e < at)) { best = v; at = e; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+                if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+            }
+            if (at >= E) at = 0;                       // (every score was NaN)
+            if (lane == k) { mine = best; mine_at = at; }
+            if (lane == (at & 31)) zr[at] = -INFINITY; // the lane that reads this place again
+        }
+        const float top_score = __shfl_sync(0xffffffffu, mine, 0);
+        const float w = lane < top ? expf(mine - top_score) : 0.0f;
+        const float sum = warp_sum(w);
+        if (lane < top) {
+            ids[(size_t)t * top + lane] = mine_at;
+            wts[(size_t)t * top + lane] = w / sum;
+        }
+        return;
+    }
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = 0x7fffffff;

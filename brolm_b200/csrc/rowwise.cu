@@ -301,7 +301,8 @@ __global__ void __launch_bounds__(256) norm_sigmoid_gate_kernel(const Y* __restr
 
 // out[t, h * hd + e] = y[t, h * hd + e] * rsqrt(mean over the head of y^2 + eps) * (w or 1) * gate(z[t, h * hd + e]);
 // gate: 0 silu, 1 sigmoid.  A warp per (token, head).  V = 4: rows, heads and addresses in steps of 16 bytes (8 for a
-// bfloat16 result), the head kept in registers up to NREG pieces a lane; V = 1: anything, read twice.
+// bfloat16 result), the head kept in registers as NREG pieces of four a lane (1: heads of up to 128, more warps an SM);
+// V = 1: anything, read twice.
 __device__ __forceinline__ float gate_of(float z, int gate) {
     const float s = 1.0f / (1.0f + expf(-z));
     return gate == 0 ? z * s : s;
@@ -316,11 +317,10 @@ __device__ __forceinline__ void store_four(bf16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = u;
 }
 
-template <typename O, int V>
+template <typename O, int V, int NREG>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ y, long ldy, const float* __restrict__ z,
                                                              long ldz, const float* __restrict__ w, float eps, int heads, int hd,
                                                              int gate, O* __restrict__ out, long ldo, int tokens) {
-    constexpr int NREG = 4;
     pdl_trigger();
     const int lane = threadIdx.x & 31;
     const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -378,15 +378,17 @@ BROLM_API int brolm_head_norm_gate(const void* y, long ldy, const void* z, long 
     const bool four = hd % 4 == 0 && hd <= 512 && ldy % 4 == 0 && ldz % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)y & 15) == 0 &&
                       ((uintptr_t)z & 15) == 0 && ((uintptr_t)out & 15) == 0;
     dim3 grid((unsigned)((units + 7) / 8));
-#define BROLM_HN(O, V) return launch_pdl(head_norm_gate_kernel<O, V>, grid, dim3(256), 0, stream, (const float*)y, ldy,   \
-                                         (const float*)z, ldz, (const float*)w, eps, heads, hd, gate, (O*)out, ldo, tokens)
+#define BROLM_HN(O, V, N) return launch_pdl(head_norm_gate_kernel<O, V, N>, grid, dim3(256), 0, stream, (const float*)y, ldy, \
+                                            (const float*)z, ldz, (const float*)w, eps, heads, hd, gate, (O*)out, ldo, tokens)
     if (out_dtype == BROLM_F32) {
-        if (four) BROLM_HN(float, 4);
-        BROLM_HN(float, 1);
+        if (four && hd <= 128) BROLM_HN(float, 4, 1);
+        if (four) BROLM_HN(float, 4, 4);
+        BROLM_HN(float, 1, 1);
     }
     if (out_dtype == BROLM_BF16) {
-        if (four) BROLM_HN(bf16, 4);
-        BROLM_HN(bf16, 1);
+        if (four && hd <= 128) BROLM_HN(bf16, 4, 1);
+        if (four) BROLM_HN(bf16, 4, 4);
+        BROLM_HN(bf16, 1, 1);
     }
 #undef BROLM_HN
     return BROLM_ERR_BAD_DTYPE;

@@ -138,7 +138,7 @@ def test_other_parts_refuse_what_they_cannot_do():
 
 
 @pytest.mark.parametrize("r", [rot(100.0, 8, (2.0, 32, 8.0, 1.0)), rot(30000.0, 12, (6.0, 512, 24.0, 1.5)),
-                                               rot(10000.0, 2, (4.0, 64, 32.0, 1.0)), rot(500.0, 6)])
+                               rot(10000.0, 2, (4.0, 64, 32.0, 1.0)), rot(500.0, 6)])
 def test_rotation_table_against_the_oracle(r):
     part = RotaryEmbedding(head_dim=16, theta=r["base"], rotary_dim=r["dims"], stretch=r.get("scaling"))
     part.prepare(700, torch.device("cpu"))

@@ -848,24 +848,24 @@ BROLM_API int brolm_gated_act(const void* gate_up, void* out, int dtype, int tok
 }
 
 // ---------------------------------------------------------------------------
-// Logits to float with the final soft-cap:  out = cap * tanh(x / cap)
+// Logits to float with the final soft-cap:  out = cap * tanh(mul * x / cap), or mul * x without a cap
 // (src/gemma2.cpp:406-412, one pass instead of three).  In and out may be the
 // same float buffer.
 // ---------------------------------------------------------------------------
 template <typename T>
-__global__ void softcap_kernel(const T* __restrict__ x, float* __restrict__ out, size_t n, float cap) {
+__global__ void softcap_kernel(const T* __restrict__ x, float* __restrict__ out, size_t n, float cap, float mul) {
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
-        out[i] = soft_cap(to_float(x[i]), cap);
+        out[i] = soft_cap(to_float(x[i]) * mul, cap);
 }
 
-BROLM_API int brolm_softcap(const void* x, int dtype, void* out, long long n, float cap, cudaStream_t stream) {
+BROLM_API int brolm_softcap(const void* x, int dtype, void* out, long long n, float cap, float mul, cudaStream_t stream) {
     if (n <= 0) return BROLM_OK;
     long long blocks = (n + 255) / 256;
     if (blocks > device_sm_count() * 32) blocks = device_sm_count() * 32;
     if (dtype == BROLM_F32)
-        softcap_kernel<float><<<(int)blocks, 256, 0, stream>>>((const float*)x, (float*)out, (size_t)n, cap);
+        softcap_kernel<float><<<(int)blocks, 256, 0, stream>>>((const float*)x, (float*)out, (size_t)n, cap, mul);
     else if (dtype == BROLM_BF16)
-        softcap_kernel<bf16><<<(int)blocks, 256, 0, stream>>>((const bf16*)x, (float*)out, (size_t)n, cap);
+        softcap_kernel<bf16><<<(int)blocks, 256, 0, stream>>>((const bf16*)x, (float*)out, (size_t)n, cap, mul);
     else
         return BROLM_ERR_BAD_DTYPE;
     return launch_status();

@@ -48,7 +48,7 @@ struct StreamArgs {
     int M, N, K;             // N: output columns (EPI_GATED: W has 2N rows, gate then up)
     int out_f32;
     int act;
-    float cap;
+    float cap, mul;
     int ksplit;
     long long part_stride;   // elements between the float partial sums of two K slices
     int row_tiles, items;
@@ -239,7 +239,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_stream_kernel(const __grid_co
                     col = rt * BR + lrow;
                     if (EPI == EPI_SOFTCAP) {
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) o[i] = soft_cap(o[i], g.cap);
+                        for (int i = 0; i < 16; ++i) o[i] = soft_cap(o[i] * g.mul, g.cap);
                     }
                 }
                 if (writer && col < g.N) {
@@ -286,11 +286,12 @@ int dispatch(const CUtensorMap& mw, const CUtensorMap& mx, const StreamArgs& g, 
 }  // namespace
 
 // epilogue 0: Y = X W^T (bfloat16 or float; with ksplit > 1 float partial sums, slice s at y + s * part_stride);
-// 1: Y = act(X Wg^T) * (X Wu^T), W = [Wg; Wu] of 2N rows, N a multiple of 64; 2: Y = cap * tanh(X W^T / cap), float.
+// 1: Y = act(X Wg^T) * (X Wu^T), W = [Wg; Wu] of 2N rows, N a multiple of 64; 2: Y = cap * tanh(mul * X W^T / cap),
+// float (cap 0: mul * X W^T).
 // M <= 128; K, ldx and ldw multiples of 8 elements; base addresses 16-byte aligned.
 BROLM_API int brolm_gemm_stream(const void* x, int ldx, const void* w, int ldw, void* y, int ldy, int M, int N, int K,
-                                int epilogue, int out_f32, int act, float cap, int ksplit, long long part_stride,
-                                cudaStream_t stream) {
+                                int epilogue, int out_f32, int act, float cap, float mul, int ksplit,
+                                long long part_stride, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return BROLM_OK;
     if (M > 128) return BROLM_ERR_TOO_LARGE;
     if (K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return BROLM_ERR_ALIGNMENT;
@@ -307,7 +308,7 @@ BROLM_API int brolm_gemm_stream(const void* x, int ldx, const void* w, int ldw, 
     if (st) return st;
     StreamArgs g;
     g.y = y; g.ldy = ldy; g.M = M; g.N = N; g.K = K; g.out_f32 = epilogue == EPI_SOFTCAP ? 1 : out_f32; g.act = act;
-    g.cap = cap; g.ksplit = ksplit; g.part_stride = part_stride;
+    g.cap = cap; g.mul = mul; g.ksplit = ksplit; g.part_stride = part_stride;
     const int out_rows = epilogue == EPI_GATED ? 64 : BR;
     g.row_tiles = (N + out_rows - 1) / out_rows;
     // slices that would be empty (K blocks do not divide evenly) are left out

@@ -341,6 +341,8 @@ struct GroupedArgs {
     int mode;
     int rows;                                 // heads: rows of every group
     int tiles_per_group;                      // heads
+    const void* gate; long ld_gate;           // heads: the result of (row, group) times sigmoid(gate[row][group]), or null
+    int gate_f32;
     const int32_t* tile_group;                // experts: the tile list of group_kernel
     const int32_t* tile_row0;
     const int32_t* offsets;
@@ -378,6 +380,11 @@ __device__ __forceinline__ int tile_rows(const GroupedArgs& g, int bt, RowInfo* 
             if (g.mode == MODE_HEADS) {
                 ri.a_off = (long)s * g.lda + (long)group * g.a_goff;
                 ri.o_off = (long)s * g.ldo + (long)group * g.o_goff;
+                if (g.gate) {
+                    const size_t at = (size_t)s * g.ld_gate + group;
+                    const float z = g.gate_f32 ? ((const float*)g.gate)[at] : to_float(((const bf16*)g.gate)[at]);
+                    ri.scale = 1.0f / (1.0f + expf(-z));
+                }
             } else {
                 const int p = g.perm[s];
                 const int tok = p / g.top, choice = p - tok * g.top;
@@ -582,7 +589,8 @@ __global__ void __launch_bounds__(128) grouped_bf16_kernel(GroupedArgs g, int ve
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) {
                 const int n = n0 + wn + nt * 8 + (lane & 3) * 2;
-                const float v0 = act_of(acc[mt][nt][2 * half], g.act), v1 = act_of(acc[mt][nt][2 * half + 1], g.act);
+                const float f = scaled ? 1.0f : ri.scale;      // (an expert's weight has met the input row)
+                const float v0 = act_of(acc[mt][nt][2 * half] * f, g.act), v1 = act_of(acc[mt][nt][2 * half + 1] * f, g.act);
                 if (g.out_f32) {
                     float* o = (float*)g.out + ri.o_off + n;
                     if (n < g.N) o[0] = v0;
@@ -814,12 +822,14 @@ BROLM_API int brolm_group_pairs(const void* ids, int pairs, int experts, void* p
 }
 
 // Per-head product: out[r, g * o_goff + n] = sum_k w[g][n][k] * a[r, g * a_goff + k], for `rows` rows and
-// `groups` heads.  Output float or the operands' type.
+// `groups` heads.  Output float or the operands' type.  gate (float or bfloat16 [rows][ld_gate], or null): the result
+// of row r and head g is multiplied by sigmoid(gate[r][g]), on the float sums.
 BROLM_API int brolm_heads_linear(int dtype, const void* a, long lda, long a_goff, const void* w, long ldw, long w_goff,
                                  void* out, long ldo, long o_goff, int out_f32, int rows, int groups, int N, int K,
-                                 cudaStream_t stream) {
+                                 const void* gate, long ld_gate, int gate_f32, cudaStream_t stream) {
     if (rows <= 0 || groups <= 0) return BROLM_OK;
     GroupedArgs g = {};
+    g.gate = gate; g.ld_gate = ld_gate; g.gate_f32 = gate_f32;
     g.a = a; g.lda = lda; g.a_goff = a_goff; g.w = w; g.ldw = ldw; g.w_goff = w_goff;
     g.out = out; g.ldo = ldo; g.o_goff = o_goff; g.out_f32 = out_f32; g.act = ACT_NONE;
     g.N = N; g.K = K; g.mode = MODE_HEADS; g.rows = rows; g.tiles_per_group = (rows + GBM - 1) / GBM;

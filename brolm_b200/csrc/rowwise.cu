@@ -6,6 +6,7 @@
 //   qkv_norm_write  RMS norm of the whole query row and of the whole key row of a token (one
 //                   statistic over all heads), and keys and values into the paged cache; the
 //                   value rows may have a size of their own
+//   table_gate      out = act(sum of the parts of z) * (a run of columns of the row that the token's id picks in a table)
 //   gate_group_norm out = rmsnorm per group of (y * silu(z)) * gain
 //   experts_combine out = sum over a token's choices of weight * (expert's result | the token's own
 //                   row for an identity expert) + the shared expert's result, the latter times
@@ -96,6 +97,24 @@ __global__ void __launch_bounds__(256) bias_act4_kernel(const float* y, int n_pa
         v[e] = row_act(v[e], act);
     }
     store4(out + (size_t)r * ldo + c, v);              // (y and out may be the same rows: a thread reads what it writes first)
+}
+
+template <typename W, typename O>
+__global__ void __launch_bounds__(256) table_gate_kernel(const float* __restrict__ z, int n_parts, long long part_stride,
+                                                         const int32_t* __restrict__ ids, const W* __restrict__ table, long ldt,
+                                                         int first, int act, O* __restrict__ out, long ldo, int tokens, int n) {
+    pdl_trigger();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    const int t = i / n, c = i - t * n;
+    const bool in = t < tokens;
+    // the table is a weight, but which row is read hangs on an id that the kernel before this one may have drawn
+    pdl_wait();
+    if (!in) return;
+    const float e = to_float(table[(size_t)ids[t] * ldt + first + c]);
+    const float* zr = z + (size_t)t * n + c;
+    float v = zr[0];
+    for (int s = 1; s < n_parts; ++s) v += zr[(size_t)s * part_stride];
+    out[(size_t)t * ldo + c] = from_float<O>(row_act(v, act) * e);
 }
 
 __global__ void __launch_bounds__(256) scaled_sum_kernel(const float* __restrict__ a, int a_parts, long long a_stride, float sa,
@@ -437,6 +456,24 @@ BROLM_API int brolm_bias_act(const void* y, int y_dtype, int n_parts, long long 
     if (y_dtype == BROLM_BF16 && bias_dtype == BROLM_BF16) BROLM_BA2(bf16, bf16);
 #undef BROLM_BA2
 #undef BROLM_BA
+    return BROLM_ERR_BAD_DTYPE;
+}
+
+// z float [n_parts][tokens][n]; ids int32 [tokens]; table [.][ldt] float or bfloat16, columns first .. first + n.
+BROLM_API int brolm_table_gate(const void* z, int n_parts, long long part_stride, const void* ids, const void* table,
+                               int table_dtype, long ldt, int first, int act, void* out, int out_dtype, long ldo, int tokens,
+                               int n, cudaStream_t stream) {
+    if (tokens <= 0) return BROLM_OK;
+    if (n <= 0 || n_parts < 1 || first < 0) return BROLM_ERR_BAD_SIZE;
+    if ((long long)tokens * n > 0x7fffff00LL) return BROLM_ERR_TOO_LARGE;
+    dim3 grid((unsigned)(((long long)tokens * n + 255) / 256));
+#define BROLM_TG(W, O) return launch_pdl(table_gate_kernel<W, O>, grid, dim3(256), 0, stream, (const float*)z, n_parts, part_stride, \
+                                         (const int32_t*)ids, (const W*)table, ldt, first, act, (O*)out, ldo, tokens, n)
+    if (table_dtype == BROLM_F32 && out_dtype == BROLM_F32) BROLM_TG(float, float);
+    if (table_dtype == BROLM_F32 && out_dtype == BROLM_BF16) BROLM_TG(float, bf16);
+    if (table_dtype == BROLM_BF16 && out_dtype == BROLM_F32) BROLM_TG(bf16, float);
+    if (table_dtype == BROLM_BF16 && out_dtype == BROLM_BF16) BROLM_TG(bf16, bf16);
+#undef BROLM_TG
     return BROLM_ERR_BAD_DTYPE;
 }
 

@@ -38,6 +38,7 @@ class StepContext:
     host_lengths: list             # host copy of kv_len
     max_kv_len: int = 0            # an upper bound of kv_len for sizing launches (a captured graph fixes it)
     ragged: bool = False           # decode: the lengths are far from equal (a hint for how attention cuts its work)
+    tokens: Optional[torch.Tensor] = None      # int32 [n_tokens], the step's token ids (set by the model's pass)
     # what one layer of a pass leaves for later layers of the same pass (by name; the model empties it
     # at the start of every pass): values that belong to the step's tokens, never to a sequence
     carry: dict = dataclasses.field(default_factory=dict)

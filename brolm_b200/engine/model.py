@@ -169,6 +169,7 @@ class DecoderModel:
             raise RuntimeError("forward: weights not loaded")
         lay = self.layout
         ctx.carry.clear()
+        ctx.tokens = tokens
         h = torch.empty((ctx.n_tokens, lay.embedding.hidden), dtype=torch.float32, device=self.device)
         emb = lay.embedding
         if emb.pairs is not None:
@@ -202,15 +203,15 @@ class DecoderModel:
             return torch.empty((0, lay.embedding.vocab), dtype=torch.float32, device=self.device)
         xf = self.final_norm.apply(h, head_in, rows=rows)
         self.last_hidden = xf            # wlejon/brolm's hidden_out (include/brolm/gemma2.h:121-125)
-        cap = float(lay.head.softcap or 0.0)
+        cap, scale = float(lay.head.softcap or 0.0), float(lay.head.scale)
         if kernels.gemm_stream_ok(xf, self.head):
             # the largest stream of weights of a decode step: the TMA ring into tcgen05, soft-cap in the epilogue
             logits = torch.empty((xf.shape[0], self.head.shape[0]), dtype=torch.float32, device=self.device)
-            kernels.gemm_stream(xf, self.head, logits, "softcap" if cap > 0 else "store", cap=cap)
+            kernels.gemm_stream(xf, self.head, logits, "softcap" if cap > 0 or scale != 1.0 else "store", cap=cap, scale=scale)
             return logits
         logits = linear(xf, self.head, out_dtype=torch.float32)
-        if cap > 0:
-            kernels.softcap(logits, logits, cap)
+        if cap > 0 or scale != 1.0:
+            kernels.softcap(logits, logits, cap, scale)
         return logits
 
 

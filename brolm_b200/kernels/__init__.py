@@ -222,11 +222,11 @@ def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str, limit: 
            "gated_act")
 
 
-def softcap(x: torch.Tensor, out: torch.Tensor, cap: float) -> None:
-    """out (float32) = cap * tanh(x / cap); cap <= 0 only converts."""
+def softcap(x: torch.Tensor, out: torch.Tensor, cap: float, scale: float = 1.0) -> None:
+    """out (float32) = cap * tanh(scale * x / cap), or scale * x with cap <= 0."""
     assert x.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32 and x.numel() == out.numel()
-    f = _fn("core", "brolm_softcap", [c_void_p, c_int, c_void_p, c_longlong, c_float, c_void_p])
-    _check(f(_ptr(x), _code(x), _ptr(out), x.numel(), cap, _stream()), "softcap")
+    f = _fn("core", "brolm_softcap", [c_void_p, c_int, c_void_p, c_longlong, c_float, c_float, c_void_p])
+    _check(f(_ptr(x), _code(x), _ptr(out), x.numel(), cap, scale, _stream()), "softcap")
 
 
 def embed_pairs(ids: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor, cu_q: torch.Tensor,
@@ -256,30 +256,47 @@ def concat_cast(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def latent_rows(proj: torch.Tensor, q_cols: int, positions: torch.Tensor, cos_sin: Optional[torch.Tensor], rotary_dim: int,
-                gain: torch.Tensor, eps: float, heads: int, dn: int, dr: int, rank: int, lat: torch.Tensor,
-                qlat: torch.Tensor, pages: Optional[torch.Tensor] = None,
-                cache_rows: Optional[torch.Tensor] = None) -> None:
-    """The row-wise step of latent attention.  ``proj`` (tokens, q_cols + rank + dr): per head [dn | dr] queries,
-    then the compressed row [rank | dr].  Writes ``lat`` (tokens, Dp) = [rmsnorm(compressed) * gain | rotated key
-    part | zeros], the same row into ``pages`` at ``cache_rows`` (negative: not kept), and the rotated query
-    parts into columns rank .. of every head of ``qlat`` (tokens, heads * Dp)."""
-    Dp = lat.shape[1]
-    assert proj.stride(1) == 1 and proj.shape[1] >= q_cols + rank + dr and q_cols == heads * (dn + dr)
-    assert lat.dtype == proj.dtype and qlat.dtype == proj.dtype and gain.dtype == proj.dtype
-    assert lat.is_contiguous() and qlat.is_contiguous() and qlat.shape == (proj.shape[0], heads * Dp)
-    assert gain.is_contiguous() and gain.numel() == rank
-    assert positions.dtype == torch.int32 and positions.numel() == proj.shape[0]
+                gain: Optional[torch.Tensor], eps: float, heads: int, dn: int, dr: int, rank: int,
+                lat: Optional[torch.Tensor], qlat: Optional[torch.Tensor], pages: Optional[torch.Tensor] = None,
+                cache_rows: Optional[torch.Tensor] = None, *, pairing: str = "half", queries: Optional[torch.Tensor] = None,
+                cq: Optional[torch.Tensor] = None, cq_gain: Optional[torch.Tensor] = None, width: Optional[int] = None) -> None:
+    """The row-wise step of latent attention, in up to three parts.  ``proj`` (tokens, .) holds the compressed row
+    [rank | dr] from column ``q_cols`` on.  ``lat`` (tokens, Dp) <- [rmsnorm(compressed) * gain | rotated key part |
+    zeros], the same row into ``pages`` at ``cache_rows`` (negative: not kept).  ``qlat`` (tokens, heads * Dp): the
+    rotated query parts go into columns rank .. of every head; the queries, per head [dn | dr], are the first columns
+    of ``proj`` or the rows of ``queries``.  ``cq`` (tokens, Q) <- rmsnorm(the first Q columns of proj) * ``cq_gain``,
+    the latent that queries of their own product come from.  A part whose result is None is left out (``width``: Dp
+    when there is no ``lat``)."""
+    Dp = lat.shape[1] if lat is not None else int(width or rank + dr)
+    assert proj.stride(1) == 1 and positions.dtype == torch.int32 and positions.numel() == proj.shape[0]
+    if pairing not in ROPE_PAIRINGS:
+        raise KernelError(f"latent_rows: unknown pairing '{pairing}' (known: {sorted(ROPE_PAIRINGS)})")
+    q_rows, Q = None, 0
+    if lat is not None:
+        assert proj.shape[1] >= q_cols + rank + dr and lat.dtype == proj.dtype and lat.is_contiguous()
+        assert gain.dtype == proj.dtype and gain.is_contiguous() and gain.numel() == rank
+    if qlat is not None:
+        q_rows = queries if queries is not None else proj
+        assert q_rows.dtype == proj.dtype and q_rows.stride(1) == 1 and q_rows.shape[1] >= heads * (dn + dr)
+        assert qlat.dtype == proj.dtype and qlat.is_contiguous() and qlat.shape == (proj.shape[0], heads * Dp)
+        assert queries is not None or lat is None or q_cols >= heads * (dn + dr)
+    if cq is not None:
+        Q = cq.shape[1]
+        assert cq.dtype == proj.dtype and cq.is_contiguous() and cq.shape[0] == proj.shape[0] and proj.shape[1] >= Q
+        assert cq_gain.dtype == proj.dtype and cq_gain.is_contiguous() and cq_gain.numel() == Q
     if cos_sin is not None:
         assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1:] == (rotary_dim // 2, 2)
     if pages is not None:
-        assert pages.dtype == proj.dtype and pages.is_contiguous() and pages.shape[-1] == Dp
+        assert pages.dtype == proj.dtype and pages.is_contiguous() and pages.shape[-1] == Dp and lat is not None
         assert cache_rows is not None and cache_rows.dtype == torch.int32 and cache_rows.numel() == proj.shape[0]
-    f = _fn("latent", "brolm_latent_rows", [c_int, c_void_p, c_long, c_int, c_void_p, c_void_p, c_int, c_void_p, c_float,
-                                            c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                                            c_int, c_void_p])
-    _check(f(_code(proj), _ptr(proj), proj.stride(0), q_cols, _ptr(positions), _ptr(cos_sin),
-             rotary_dim if cos_sin is not None else 0, _ptr(gain), eps, heads, dn, dr, rank, Dp, _ptr(lat), _ptr(qlat),
-             _ptr(pages), _ptr(cache_rows) if pages is not None else None, proj.shape[0], _stream()), "latent_rows")
+    f = _fn("latent", "brolm_latent_rows", [c_int, c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_int, c_void_p, c_void_p,
+                                            c_void_p, c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_int, c_int, c_int,
+                                            c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+    _check(f(_code(proj), _ptr(proj), proj.stride(0), q_cols, _ptr(q_rows), q_rows.stride(0) if q_rows is not None else 0, 0, Q,
+             _ptr(cq_gain) if cq is not None else None, _ptr(cq), _ptr(positions), _ptr(cos_sin),
+             rotary_dim if cos_sin is not None else 0, ROPE_PAIRINGS[pairing], _ptr(gain) if lat is not None else None, eps,
+             heads, dn, dr, rank, Dp, _ptr(lat), _ptr(qlat), _ptr(pages), _ptr(cache_rows) if pages is not None else None,
+             proj.shape[0], _stream()), "latent_rows")
 
 
 ROUTE_MODES = {"logistic": 0, "softmax": 1, "softmax_chosen": 2}
@@ -425,8 +442,10 @@ def grouped_tc_status(reset: bool = False) -> int:
     return f(1 if reset else 0)
 
 
-def heads_linear(a: torch.Tensor, a_head: int, weight: torch.Tensor, out: torch.Tensor, o_head: int) -> None:
+def heads_linear(a: torch.Tensor, a_head: int, weight: torch.Tensor, out: torch.Tensor, o_head: int,
+                 gate: Optional[torch.Tensor] = None) -> None:
     """A product per head: out[t, h * o_head + n] = sum_k weight[h, n, k] * a[t, h * a_head + k].
+    ``gate`` (tokens, heads) logits: head h's result of token t is multiplied by sigmoid(gate[t, h]), on the float sums.
     ``weight`` [heads, N, K]; a and out are packed rows whose heads lie ``a_head`` / ``o_head`` apart (a head's
     slice may be wider than K or N).  float32 everywhere, or bfloat16 operands with a bfloat16 or float32 result."""
     H, N, K = weight.shape
@@ -434,10 +453,14 @@ def heads_linear(a: torch.Tensor, a_head: int, weight: torch.Tensor, out: torch.
     assert a.shape[0] == out.shape[0] and K <= a_head and N <= o_head
     assert (H - 1) * a_head + K <= a.shape[1] and (H - 1) * o_head + N <= out.shape[1]
     assert out.dtype in (torch.float32, a.dtype)
+    if gate is not None:
+        assert gate.shape == (a.shape[0], H) and gate.stride(1) == 1
     f = _fn("grouped", "brolm_heads_linear", [c_int, c_void_p, c_long, c_long, c_void_p, c_long, c_long, c_void_p, c_long,
-                                              c_long, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                              c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long, c_int, c_void_p])
     _check(f(_code(a), _ptr(a), a.stride(0), a_head, _ptr(weight), K, N * K, _ptr(out), out.stride(0), o_head,
-             1 if out.dtype == torch.float32 else 0, a.shape[0], H, N, K, _stream()), "heads_linear")
+             1 if out.dtype == torch.float32 else 0, a.shape[0], H, N, K, _ptr(gate),
+             gate.stride(0) if gate is not None else 0, 1 if gate is not None and _code(gate) == F32 else 0, _stream()),
+           "heads_linear")
 
 
 EXPERT_ACTS = {"none": 0, "relu2": 1}
@@ -650,6 +673,53 @@ def residual_group_rmsnorm(h: torch.Tensor, y: torch.Tensor, post_weight: Option
              _ptr(next_weight), next_eps, next_offset, _CODES[wd] if wd is not None else F32,
              _ptr(out) if out is not None else None, _code(out) if out is not None else F32, h.shape[0], h.shape[-1],
              groups, _stream()), "residual_group_rmsnorm")
+
+
+def layernorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+              rows: Optional[torch.Tensor] = None) -> None:
+    """out[r] = (x - mean(x)) * rsqrt(mean((x - mean(x))^2) + eps) * weight for x[rows[r] or r], float32 rows."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and weight.is_contiguous()
+    n, hidden = out.shape[0], x.shape[-1]
+    assert weight.numel() == hidden and out.shape[-1] == hidden
+    if rows is not None:
+        assert rows.dtype == torch.int32 and rows.numel() == n
+    else:
+        assert x.shape[0] == n
+    f = _fn("layernorm", "brolm_layernorm", [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int,
+                                             c_void_p])
+    _check(f(_ptr(x), _ptr(rows), _ptr(weight), _code(weight), eps, _ptr(out), _code(out), n, hidden, _stream()), "layernorm")
+
+
+def residual_layernorm(h: torch.Tensor, y: torch.Tensor, post_weight: Optional[torch.Tensor], post_eps: float,
+                       post_offset: float, next_weight: torch.Tensor, next_eps: float, out: torch.Tensor) -> None:
+    """h += rmsnorm(y; post) (or y when post_weight is None); out = layernorm(h; next).
+    ``y`` float32, may be [parts, rows, hidden]: partial sums that are added in order first."""
+    assert h.dtype == torch.float32 and y.dtype == torch.float32 and h.is_contiguous() and y.is_contiguous()
+    assert tuple(y.shape[-2:]) == tuple(h.shape) and out.is_contiguous() and out.shape == h.shape
+    n_parts, part_stride = (y.shape[0], y.stride(0)) if y.dim() == 3 else (1, 0)
+    for w in (post_weight, next_weight):
+        assert w is None or (w.is_contiguous() and w.numel() == h.shape[-1])
+    if post_weight is not None and post_weight.dtype != next_weight.dtype:
+        raise KernelError("residual_layernorm: both gains must have one element type")
+    f = _fn("layernorm", "brolm_residual_layernorm", [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_float, c_float, c_void_p,
+                                                      c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(h), _ptr(y), n_parts, part_stride, _ptr(post_weight), post_eps, post_offset, _ptr(next_weight),
+             _code(next_weight), next_eps, _ptr(out), _code(out), h.shape[0], h.shape[-1], _stream()), "residual_layernorm")
+
+
+def table_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, first: int, activation: str, out: torch.Tensor) -> None:
+    """out[t, i] = act(z[t, i]) * table[ids[t], first + i]; z float32 (tokens, n), or [parts, tokens, n] partial sums."""
+    tokens, n = out.shape
+    assert z.dtype == torch.float32 and z.is_contiguous() and tuple(z.shape[-2:]) == (tokens, n) and out.stride(1) == 1
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() == tokens
+    assert table.stride(1) == 1 and 0 <= first and first + n <= table.shape[1]
+    if activation not in ROW_ACTS:
+        raise KernelError(f"table_gate: unknown activation '{activation}' (known: {sorted(ROW_ACTS)})")
+    n_parts, part_stride = (z.shape[0], z.stride(0)) if z.dim() == 3 else (1, 0)
+    f = _fn("rowwise", "brolm_table_gate", [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_long, c_int, c_int, c_void_p,
+                                            c_int, c_long, c_int, c_int, c_void_p])
+    _check(f(_ptr(z), n_parts, part_stride, _ptr(ids), _ptr(table), _code(table), table.stride(0), first, ROW_ACTS[activation],
+             _ptr(out), _code(out), out.stride(0), tokens, n, _stream()), "table_gate")
 
 
 def gate_group_norm(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, eps: float, groups: int,
@@ -889,6 +959,55 @@ def decay_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
     _check(f(_ptr(qkv), _code(qkv), qkv.stride(0), q_off, k_off, v_off, heads, dim, v_dim, SCAN_ACTS[activation],
              _ptr(decay_m1), *_seq(cu_q, kv_len, slots, state), _ptr(out), out.stride(0), batch, int(max_q_len),
              _ptr(cos_sin), rot, float(k_scale), _stream()), "decay_scan")
+
+
+DELTA_NORM_EPS = 1e-6       # under the root of the unit vectors of q and k
+
+
+def delta_rows(proj: torch.Tensor, taps: torch.Tensor, n_kv: int, dim: int, heads: int, v_dim: int, q_scale: float,
+               a_log: torch.Tensor, dt_bias: torch.Tensor, tok_seq: torch.Tensor, positions: torch.Tensor, cu_q: torch.Tensor,
+               kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, tail_off: int, move_tail: bool,
+               u: torch.Tensor, gates: torch.Tensor, qk: torch.Tensor, norm_eps: float = DELTA_NORM_EPS) -> None:
+    """The gated delta rule's inputs from a projection row [q: n_kv * dim | k: n_kv * dim | v: heads * v_dim | heads
+    logits of beta | heads step sizes], all float32: q, k and v after a causal convolution (``taps`` float32 [K, C], row
+    K - 1 the token's own) and silu, q and k as unit vectors per head (q times ``q_scale``), into ``u`` (tokens, C);
+    ``gates`` [tokens, heads, 2] = (decay - 1, beta); ``qk`` [tokens, n_kv] = q . k.  Earlier inputs come from the K - 1
+    rows that ``state[slot, tail_off:]`` keeps; ``move_tail`` (only when every sequence brings one token) moves them on,
+    otherwise ``conv_tail`` does afterwards."""
+    K, C = taps.shape
+    T = proj.shape[0]
+    assert C == 2 * n_kv * dim + heads * v_dim and taps.dtype == torch.float32 and taps.is_contiguous()
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= C + 2 * heads
+    assert u.dtype == torch.float32 and u.stride(1) == 1 and u.shape == (T, C) and tail_off + (K - 1) * C <= state.shape[1]
+    assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.numel() == T * heads * 2
+    assert qk.dtype == torch.float32 and qk.is_contiguous() and qk.numel() == T * n_kv
+    assert tok_seq.dtype == torch.int32 and positions.dtype == torch.int32 and positions.numel() == T
+    for v in (a_log, dt_bias):
+        assert v.dtype == torch.float32 and v.is_contiguous() and v.numel() == heads
+    f = _fn("delta_rule", "brolm_delta_rows", [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                               c_long, c_long, c_int, c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p])
+    _check(f(_ptr(proj), proj.stride(0), _ptr(taps), K, n_kv, dim, heads, v_dim, norm_eps, q_scale, _ptr(a_log), _ptr(dt_bias),
+             _ptr(tok_seq), _ptr(positions), *_seq(cu_q, kv_len, slots, state), tail_off, 1 if move_tail else 0, _ptr(u),
+             u.stride(0), _ptr(gates), _ptr(qk), T, _stream()), "delta_rows")
+
+
+def delta_scan(u: torch.Tensor, gates: torch.Tensor, qk: torch.Tensor, n_kv: int, dim: int, heads: int, v_dim: int,
+               cu_q: torch.Tensor, kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+               batch: int, max_q_len: int = 0) -> None:
+    """The gated delta rule over the packed tokens, on what ``delta_rows`` made: per head S <- g S, w = beta (v - S^T k),
+    S <- S + k w^T, out = S^T q.  S is the first ``decay_state_size(heads, dim, v_dim)`` floats of ``state[slot]``.
+    ``max_q_len`` 1 says that every sequence brings one token; 0: unknown."""
+    T = u.shape[0]
+    assert u.dtype == torch.float32 and u.stride(1) == 1 and u.shape[1] == 2 * n_kv * dim + heads * v_dim
+    assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.numel() == T * heads * 2
+    assert qk.dtype == torch.float32 and qk.is_contiguous() and qk.numel() == T * n_kv
+    assert out.dtype == torch.float32 and out.stride(1) == 1 and out.shape == (T, heads * v_dim)
+    assert state.shape[1] >= decay_state_size(heads, dim, v_dim)
+    f = _fn("delta_rule", "brolm_delta_scan", [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                                               c_void_p, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_void_p])
+    _check(f(_ptr(u), u.stride(0), _ptr(gates), _ptr(qk), n_kv, dim, heads, v_dim, *_seq(cu_q, kv_len, slots, state), _ptr(out),
+             out.stride(0), batch, int(max_q_len), _stream()), "delta_scan")
 
 
 def rotate_heads(rows: torch.Tensor, q_off: int, k_off: int, heads: int, dim: int, positions: torch.Tensor,
@@ -1190,11 +1309,12 @@ def gemm_stream_parts(x: torch.Tensor, weight: torch.Tensor, sms: Optional[int] 
 
 
 def gemm_stream(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: str = "store",
-                activation: str = "gelu_tanh", cap: float = 0.0, limit: float = 0.0) -> None:
+                activation: str = "gelu_tanh", cap: float = 0.0, limit: float = 0.0, scale: float = 1.0) -> None:
     """out = x @ weight^T for at most 128 rows of x on tcgen05, the weights streamed through a TMA ring.
 
     ``epilogue``: "store" (out bfloat16 or float32, or [parts, M, N] float32 partial sums of K slices),
-    "gated" (weight = [Wg; Wu], out = act(x Wg^T) * (x Wu^T), width a multiple of 64), "softcap" (float32)."""
+    "gated" (weight = [Wg; Wu], out = act(x Wg^T) * (x Wu^T), width a multiple of 64), "softcap"
+    (float32, cap * tanh(scale * . / cap), or scale * . without a cap)."""
     assert gemm_stream_ok(x, weight) and out.stride(-1) == 1 and out.shape[-2] == x.shape[0]
     M, K = x.shape
     code = {"store": 0, "gated": 1, "softcap": 2}[epilogue]
@@ -1206,12 +1326,13 @@ def gemm_stream(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilog
         ksplit, part_stride = out.shape[0], out.stride(0)
     if code == 2:
         assert out.dtype == torch.float32
+    assert scale == 1.0 or code == 2
     if activation not in ACTIVATIONS:
         raise KernelError(f"gemm_stream: unknown activation '{activation}'")
     f = _fn("gemm_stream", "brolm_gemm_stream", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                                                 c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p])
+                                                 c_int, c_int, c_int, c_float, c_float, c_int, c_longlong, c_void_p])
     _check(f(_ptr(x), x.stride(0), _ptr(weight), weight.stride(0), _ptr(out), out.stride(-2), M, N, K, code,
-             1 if out.dtype == torch.float32 else 0, ACTIVATIONS[activation], limit if code == 1 else cap, ksplit,
+             1 if out.dtype == torch.float32 else 0, ACTIVATIONS[activation], limit if code == 1 else cap, scale, ksplit,
              part_stride, _stream()), "gemm_stream")
 
 
@@ -1577,4 +1698,4 @@ __all__ = ["KernelBuildError", "KernelError", "build_all", "launch_count", "devi
            "rope_kv_write", "rope_kv_write_parts", "gated_act", "softcap", "linear_f32", "skinny_gemm", "skinny_qkv_rope", "skinny_ok", "skinny_parts", "skinny_rope_tiles", "gemm_tc", "gemm_tc2", "gemm_tc2_status", "gemm_tc_ok", "gemm_tc_status", "gemm_stream", "gemm_stream_ok", "gemm_stream_parts", "stream_rows",
            "gemm_stream_status", "attention_simt", "attention_prefill_mma", "attention_prefill_tc", "attention_prefill_tc_ok", "attention_prefill_tc_split", "attention_tc_status", "attention_decode_mma",
            "decode_splits", "argmax", "sample", "cast", "bias_act", "scaled_sum", "qkv_norm_write", "gate_group_norm", "head_norm_gate", "rotate_heads",
-           "experts_combine", "causal_conv", "conv_tail", "gated_scan", "ssm_scan", "block_matvec_f32", "block_matvec_ok", "split_halves"]
+           "layernorm", "residual_layernorm", "table_gate", "delta_rows", "delta_scan", "experts_combine", "causal_conv", "conv_tail", "gated_scan", "ssm_scan", "block_matvec_f32", "block_matvec_ok", "split_halves"]

@@ -50,6 +50,8 @@ LIBRARIES: dict[str, list[str]] = {
     "attn_headmix": ["attn_headmix.cu"],
     "groupnorm": ["groupnorm.cu"],
     "linear_attn": ["linear_attn.cu"],
+    "layernorm": ["layernorm.cu"],
+    "delta_rule": ["delta_rule.cu"],
 }
 HEADERS = ["common.cuh", "attn_mma.cuh", "attn_decode_noalloc.h", "tcgen05.cuh"]
 

@@ -95,6 +95,30 @@ class Block(Part):
 register_part("block", "sandwich", Block)
 
 
+class SideInputBlock(Block):
+    """The sandwich with a third sublayer, which reads the residual stream itself and whose result is normed before it
+    joins: x = pre_mixer(h), h += mixer(x);  x = pre_ffn(h), h += ffn(x) (may be absent);  h += post_side(side(h)).
+    ``entry`` is the part that hands ``side`` the stream in the step's element type (the ``cast`` norm)."""
+
+    kind = "block"
+
+    def __init__(self, side: Part, entry: Part, post_side_norm: Optional[Part] = None, **parts):
+        super().__init__(**parts)
+        self.side, self.entry, self.post_side_norm = side, entry, post_side_norm
+
+    def parts(self) -> dict[str, Optional[Part]]:
+        return {**super().parts(), "side": self.side, "entry": self.entry, "post_side_norm": self.post_side_norm}
+
+    def forward(self, h: torch.Tensor, x: torch.Tensor, ctx, entry, writes_cache: bool,
+                next_norm: Optional[Part]) -> Optional[torch.Tensor]:
+        x = super().forward(h, x, ctx, entry, writes_cache, self.entry)
+        y = self.side.forward(x, ctx)
+        return add_then_norm(h, y, self.post_side_norm, next_norm, ctx.dtype)
+
+
+register_part("block", "sandwich_side", SideInputBlock)
+
+
 class ParallelBlock(Part):
     """h += mixer(n1(h)) + ffn(n2(h)): both sublayers read the same stream, each through a norm of its own,
     and the stream takes both results at once.  Without a feed-forward it is h += mixer(n1(h)).  With

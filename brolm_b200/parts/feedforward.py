@@ -98,3 +98,38 @@ class DenseFeedForward(Part):
 
 
 register_part("feedforward", "dense", DenseFeedForward)
+
+
+class TokenSide(Part):
+    """A layer's input of its own per token: proj(act(gate(x)) * e), e being ``dim`` numbers of the row that the token's
+    id picks in a table shared by all layers, those from ``first`` on.  No bias; ``gate`` is (dim, hidden), ``proj``
+    (hidden, dim), ``table`` (vocab, table_cols)."""
+
+    kind = "feedforward"
+    graph_safe = True
+
+    def __init__(self, hidden: int, dim: int, vocab: int, table_cols: int, first: int, activation: str = "gelu_tanh"):
+        if activation not in kernels.ROW_ACTS:
+            raise ValueError(f"token side: unknown activation '{activation}'")
+        if first < 0 or first + dim > table_cols:
+            raise ValueError("token side: the layer's part lies outside the table's rows")
+        self.hidden, self.dim, self.vocab, self.table_cols = hidden, dim, vocab, table_cols
+        self.first, self.activation = first, activation
+
+    def param_specs(self):
+        return {"gate": ParamSpec((self.dim, self.hidden)), "proj": ParamSpec((self.hidden, self.dim)),
+                "table": ParamSpec((self.vocab, self.table_cols), "table")}
+
+    def bind(self, params):
+        self.w_gate, self.w_proj, self.table = params["gate"], params["proj"], params["table"]
+        self.params = {}
+
+    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+        """x (tokens, hidden) -> (tokens, hidden) float32 (or partial sums)."""
+        z = linear(x, self.w_gate, out_dtype=torch.float32, parts_ok=True)
+        g = torch.empty((x.shape[0], self.dim), dtype=ctx.dtype, device=x.device)
+        kernels.table_gate(z, ctx.tokens, self.table, self.first, self.activation, g)
+        return linear(g, self.w_proj, out_dtype=torch.float32, parts_ok=True)
+
+
+register_part("feedforward", "token_side", TokenSide)

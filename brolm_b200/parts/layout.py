@@ -46,6 +46,7 @@ class HeadSpec:
     tensor: str                       # checkpoint name of the output matrix, (vocab, hidden)
     tied_to: Optional[str] = None     # used when ``tensor`` is absent from the checkpoint
     softcap: float = 0.0              # cap * tanh(logits / cap); 0 switches it off
+    scale: float = 1.0                # multiplies the logits (ahead of a cap)
 
 
 @dataclasses.dataclass

@@ -57,6 +57,32 @@ class RMSNorm(Part):
 register_part("norm", "rmsnorm", RMSNorm)
 
 
+class LayerNorm(Part):
+    """y = (x - mean(x)) * rsqrt(mean((x - mean(x))^2) + eps) * w, no bias.  Float arithmetic over float32 rows."""
+
+    kind = "norm"
+    graph_safe = True
+
+    def __init__(self, size: int, eps: float):
+        self.size, self.eps = size, float(eps)
+
+    def param_specs(self):
+        return {"weight": ParamSpec((self.size,), "vector")}
+
+    @property
+    def weight(self) -> torch.Tensor:
+        return self.params["weight"]
+
+    def apply(self, x: torch.Tensor, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        n = rows.numel() if rows is not None else x.shape[0]
+        out = torch.empty((n, self.size), dtype=out_dtype, device=x.device)
+        kernels.layernorm(x, self.weight, self.eps, out, rows)
+        return out
+
+
+register_part("norm", "layernorm", LayerNorm)
+
+
 class Cast(Part):
     """No norm at all: the rows as they are, in the element type asked for.  It stands where an arrangement
     whose sublayers read the residual stream itself needs an entry "norm"; in float32 the stream is handed
@@ -85,10 +111,16 @@ def add_then_norm(h: torch.Tensor, y: torch.Tensor, post: Optional[Part], nxt: O
                   out_dtype: torch.dtype) -> Optional[torch.Tensor]:
     """h += post(y) (or y);  return nxt(h) when ``nxt`` is given.
 
-    h is the float32 residual stream and is updated in place.  Two RMSNorms
-    run in one kernel with the sum; any other norm part is applied through its
+    h is the float32 residual stream and is updated in place.  Two RMSNorms, or a LayerNorm
+    behind one or none, run in one kernel with the sum; any other norm part is applied through its
     own ``apply`` and only the sum stays fused.
     """
+    if isinstance(nxt, LayerNorm) and y.dtype == torch.float32 and \
+            (post is None or (isinstance(post, RMSNorm) and post.groups == 1 and post.weight.dtype == nxt.weight.dtype)):
+        out = torch.empty(h.shape, dtype=out_dtype, device=h.device)
+        kernels.residual_layernorm(h, y, post.weight if post is not None else None, post.eps if post is not None else 0.0,
+                                   post.offset if post is not None else 0.0, nxt.weight, nxt.eps, out)
+        return out
     fused_post = post is None or isinstance(post, RMSNorm)
     plain_next = isinstance(nxt, Cast)          # no norm ahead of the next block: it wants the stream itself
     fused_next = nxt is None or plain_next or isinstance(nxt, RMSNorm)

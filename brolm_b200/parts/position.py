@@ -25,12 +25,23 @@ class RotaryEmbedding(Part):
     0), hi = min(ceil(n(slow)), rot - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), frequency i becomes
     f_i / factor * r_i + f_i (1 - r_i), and cos and sin are both multiplied by 0.1 ln(factor) + 1 (the table holds
     the products, so whoever rotates with it needs to know nothing of this).
+
+    ``bands`` = {factor, low, high, original} scales by wavelength instead, as Llama 3.1 does: with l = 2 pi / f,
+    frequencies of l < original / high stay, those of l > original / low are divided by factor, and between the two
+    s = (original / l - low) / (high - low) makes (1 - s) f / factor + s f.
     """
 
     kind = "position"
 
     def __init__(self, head_dim: int, theta: float, rotary_dim: Optional[int] = None, pairing: str = "half",
-                 stretch: Optional[dict] = None):
+                 stretch: Optional[dict] = None, bands: Optional[dict] = None):
+        if bands is not None:
+            missing = [k for k in ("factor", "low", "high", "original") if k not in bands]
+            if missing or any(not float(bands[k]) > 0 for k in ("factor", "low", "high", "original")):
+                raise ValueError(f"rotary: bands needs a positive factor, low, high and original (missing: {missing})")
+            if stretch is not None:
+                raise ValueError("rotary: stretch and bands are two ways to scale the frequencies; give one")
+        self.bands = dict(bands) if bands is not None else None
         if stretch is not None:
             missing = [k for k in ("factor", "original", "fast", "slow") if k not in stretch]
             if missing or not float(stretch["factor"]) > 0:
@@ -69,6 +80,13 @@ class RotaryEmbedding(Part):
             ramp = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
             inv_freq = inv_freq / factor * ramp + inv_freq * (1.0 - ramp)
             magnitude = 0.1 * math.log(factor) + 1.0
+        if self.bands is not None:
+            factor, low, high, original = (float(self.bands[k]) for k in ("factor", "low", "high", "original"))
+            wave = 2.0 * math.pi / inv_freq
+            share = (original / wave - low) / (high - low) if high != low else torch.zeros_like(wave)
+            blend = (1.0 - share) * inv_freq / factor + share * inv_freq
+            inv_freq = torch.where(wave < original / high, inv_freq,
+                                   torch.where(wave > original / low, inv_freq / factor, blend))
         ang = torch.arange(max_positions, dtype=torch.float64)[:, None] * inv_freq[None, :]
         self.table = (torch.stack([ang.cos(), ang.sin()], dim=-1) * magnitude).to(torch.float32).contiguous().to(device)
 

@@ -1,7 +1,8 @@
-"""Mixers that carry a state of fixed size from token to token: a gated diagonal recurrence
-and a selective state space, each behind a short causal convolution.
+"""Mixers that carry a state of fixed size from token to token: a gated diagonal recurrence,
+a selective state space and a gated delta rule, each behind a short causal convolution, and linear attention
+with a fixed decay.
 
-Both keep, per sequence, one float32 row of a state group: the recurrence's state first, then the
+All keep, per sequence, one float32 row of a state group: the recurrence's state first, then the
 convolution's last ``taps - 1`` inputs (zeros before the sequence's start).  The row is zero when a slot is
 taken, read at the start of a sequence's tokens in a step and written at their end; the same kernels serve
 a prompt and a decode step, and nothing is read back to the host.
@@ -291,6 +292,94 @@ class DecayLinearAttention(Part):
 
 
 register_part("mixer", "decay_attention", DecayLinearAttention)
+
+
+class GatedDeltaRule(Part):
+    """The gated delta rule (Yang et al., "Gated Delta Networks: Improving Mamba2 with Delta Rule").
+
+    q = W_q x and k = W_k x (``kv_heads`` x ``dim``), v = W_v x (``heads`` x ``v_dim``), each through a causal
+    convolution per channel over time (``taps`` taps, no bias) and silu; q and k are made unit vectors per head and q is
+    multiplied by dim^(-1/2); value head h works with q/k head h // (heads / kv_heads).  Per head, with
+    beta = sigmoid(W_b x) and g = exp(-exp(A_log) softplus(W_a x + dt_bias)):
+
+        S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+
+    Every head's o is divided by its own root mean square, times a gain of ``v_dim`` numbers for all heads (``norm``),
+    times silu(W_g x), then W_o.  The projection's sums and everything up to the last product's input are float32 in
+    every mode; S and the convolutions' last taps - 1 inputs are a state row per sequence, zero at the sequence's
+    start."""
+
+    kind = "mixer"
+    graph_safe = True
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, v_dim: int, taps: int, eps: float):
+        if heads % kv_heads:
+            raise ValueError("delta rule: heads must be a multiple of kv_heads")
+        if taps < 1:
+            raise ValueError("delta rule: the convolution needs at least one tap")
+        if dim > 512:
+            raise ValueError("delta rule: more than 512 query/key entries per head are beyond the kernel")
+        self.hidden, self.heads, self.kv_heads, self.dim, self.v_dim = hidden, heads, kv_heads, dim, v_dim
+        self.taps, self.eps = taps, float(eps)
+        self.qk_cols, self.v_cols = kv_heads * dim, heads * v_dim
+        self.conv_cols = 2 * self.qk_cols + self.v_cols
+        # the gate's columns of the projection start at a multiple of four, so that its rows can be read four at a time
+        self.gate_from = (self.conv_cols + 2 * heads + 3) // 4 * 4
+        self.tail_off = kernels.decay_state_size(heads, dim, v_dim)
+
+    def param_specs(self):
+        W, K = self.hidden, self.taps
+        return {"q": ParamSpec((self.qk_cols, W)), "q_conv": ParamSpec((self.qk_cols, K), "vector"),
+                "k": ParamSpec((self.qk_cols, W)), "k_conv": ParamSpec((self.qk_cols, K), "vector"),
+                "v": ParamSpec((self.v_cols, W)), "v_conv": ParamSpec((self.v_cols, K), "vector"),
+                "b": ParamSpec((self.heads, W)), "a": ParamSpec((self.heads, W)), "A_log": ParamSpec((self.heads,), "vector"),
+                "dt_bias": ParamSpec((self.heads,), "vector"), "g": ParamSpec((self.v_cols, W)),
+                "norm": ParamSpec((self.v_dim,), "vector"), "o": ParamSpec((W, self.v_cols))}
+
+    def bind(self, params):
+        names = ("q", "k", "v", "b", "a", "g")
+        kinds = {params[n].dtype for n in names}
+        dt = torch.float32 if (len(kinds) > 1 or torch.float32 in kinds) else next(iter(kinds))
+        # one product: rows [Wq; Wk; Wv; Wb; Wa; (rows of zeros up to a multiple of four); Wg]
+        rows = [params[n].to(dt) for n in names]
+        pad = self.gate_from - self.conv_cols - 2 * self.heads
+        if pad:
+            rows.insert(5, torch.zeros((pad, self.hidden), dtype=dt, device=rows[0].device))
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+        self.w_o = params["o"]
+        # tap by tap, so that neighbouring channels lie next to one another
+        self.conv = torch.cat([params[n + "_conv"].float() for n in ("q", "k", "v")], dim=0).t().contiguous()
+        self.a_log, self.dt_bias = _f32(params["A_log"]), _f32(params["dt_bias"])
+        self.gain = _f32(params["norm"]).repeat(self.heads).contiguous()
+        self.params = {}
+
+    def cache_spec(self):
+        # S, then taps - 1 rows of inputs; a row of the state group is a whole number of 16-byte pieces
+        n = self.tail_off + (self.taps - 1) * self.conv_cols
+        return StateSpec(((n + 3) // 4 * 4,), torch.float32)
+
+    def forward(self, x: torch.Tensor, ctx, entry, writes_cache: bool = True) -> torch.Tensor:
+        """x (tokens, hidden) -> (tokens, hidden) float32, or partial sums [parts, tokens, hidden]."""
+        if not writes_cache:
+            raise NotImplementedError("a mixer with a state cannot run on another layer's state")
+        T, dev = x.shape[0], x.device
+        f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
+        seq = (ctx.cu_q, ctx.kv_len, ctx.slots_dev, ctx.state(entry))
+        sizes = (self.kv_heads, self.dim, self.heads, self.v_dim)
+        single = ctx.max_q_len == 1
+        proj = linear(x, self.w_in, out_dtype=torch.float32)              # [ q | k | v | b | a | gate logits ]
+        u, gates, qk, y = f32(T, self.conv_cols), f32(T, self.heads, 2), f32(T, self.kv_heads), f32(T, self.v_cols)
+        kernels.delta_rows(proj, self.conv, *sizes, self.dim ** -0.5, self.a_log, self.dt_bias, ctx.tok_seq, ctx.positions,
+                           *seq, self.tail_off, single, u, gates, qk)
+        if not single and self.taps > 1:
+            kernels.conv_tail(proj[:, :self.conv_cols], None, self.taps, *seq, self.tail_off, ctx.batch)
+        kernels.delta_scan(u, gates, qk, *sizes, *seq, y, ctx.batch, ctx.max_q_len)
+        out = torch.empty((T, self.v_cols), dtype=ctx.dtype, device=dev)
+        kernels.head_norm_gate(y, proj[:, self.gate_from:], self.gain, self.eps, self.heads, "silu", out)
+        return linear(out, self.w_o, out_dtype=torch.float32, parts_ok=True)
+
+
+register_part("mixer", "gated_delta_rule", GatedDeltaRule)
 
 
 class SideBySide(Part):

@@ -34,6 +34,11 @@ shared expert), built to the same width, heads, experts and layer count.
 reads the other's keys and values; routed experts with a clamped gate) beside the closest design the library has,
 Ritirax, with two lightning and two attention layers of the same sizes and experts.
 
+``--arch papusun [--size s|m]``: the Papusun design (attention beside a gated delta rule, windowed latent attention of which
+one layer reads another's latents, an input per token and layer) beside the closest design the library has, Ritirax, with
+an attention, a lightning and a latent layer for each pair of its layers, of the same sizes and with feed-forwards of as
+many weights.
+
 More than one GPU is not what this library does: ``--gpus N`` with N > 1 says
 so and exits with 2.
 """
@@ -790,6 +795,141 @@ def relulix_main(args, pk) -> int:
     return 0
 
 
+# --arch papusun: a parallel and a latent layer, twice, the second latent layer reading the first one's latents; beside
+# Ritirax with an attention, a lightning and a latent layer for each pair (only two of three with a feed-forward, whose two
+# matrices hold as many weights as the gated one's three).  At m the value heads have a size of their own.
+PAPUSUN_SIZES = {
+    "s": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, d_heads=16, d_kv=16, d_dim=128, d_vdim=128, conv=4,
+              lat_heads=16, lat_dim=64, lat_rot=64, lat_vdim=64, q_rank=768, kv_rank=192, window=1024, ff=4096, side=128,
+              vocab=32768),
+    "m": dict(width=3072, heads=24, kv_heads=4, dim=128, vdim=192, d_heads=24, d_kv=8, d_dim=128, d_vdim=128, conv=4,
+              lat_heads=16, lat_dim=128, lat_rot=64, lat_vdim=128, q_rank=1024, kv_rank=192, window=1024, ff=8192, side=256,
+              vocab=65536),
+}
+
+
+def papusun_main(args, pk) -> int:
+    import torch
+
+    import brolm_b200 as bb
+
+    name = args.size if args.size in PAPUSUN_SIZES else "s"
+    z = PAPUSUN_SIZES[name]
+    dev = "cuda:0"
+    torch.cuda.set_device(0)
+    W, H, G, d, dv, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["ff"]
+    DH, DG, dd, ddv = z["d_heads"], z["d_kv"], z["d_dim"], z["d_vdim"]
+    mlp = dict(kind="dense", ff=ff)
+    left = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=d ** -0.5, softcap=30.0,
+                rot=dict(base=10000.0, dims=d, scaling=dict(factor=8.0, low=1.0, high=4.0, original=1024)))
+    right = dict(heads=DH, kv_heads=DG, dim=dd, vdim=ddv, conv=z["conv"])
+    pair = dict(left=left, right=right, left_scale=1.0, right_scale=1.0)
+    lat = dict(heads=z["lat_heads"], dim=z["lat_dim"], rot_dim=z["lat_rot"], vdim=z["lat_vdim"], q_rank=z["q_rank"],
+               kv_rank=z["kv_rank"], scale=(z["lat_dim"] + z["lat_rot"]) ** -0.5, mask=dict(size=z["window"]),
+               rot=dict(base=10000.0, dims=z["lat_rot"]))
+    layers = [dict(type="parallel", mixer=pair, mlp=mlp), dict(type="latent_attention", mixer=lat, mlp=mlp),
+              dict(type="parallel", mixer=pair, mlp=mlp), dict(type="latent_attention", mixer=dict(lat, kv_from=1), mlp=mlp)]
+    xcfg = bb.PapusunConfig.from_dict(dict(architecture="Papusun", vocab=z["vocab"], width=W, layers=layers, norm=dict(eps=1e-5),
+                                           token_side=dict(dim=z["side"]), logit_scale=0.5))
+    cmlp = dict(kind="dense", ff=ff * 3 // 2)
+    cattn = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=d ** -0.5, softcap=30.0, bias_max=128, bias_rows=32)
+    light = dict(heads=DH, dim=dd, vdim=ddv, decay=[1.0 - 2.0 ** (-3.0 - 7.0 * h / max(DH - 1, 1)) for h in range(DH)])
+    clat = {k: lat[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot")}
+    clayers = [dict(type="attention", mixer=cattn, mlp=None), dict(type="lightning", mixer=light, mlp=cmlp),
+               dict(type="latent_attention", mixer=clat, mlp=cmlp)] * 2
+    ccfg = bb.RitiraxConfig.from_dict(dict(architecture="Ritirax", vocab=z["vocab"], width=W, layers=clayers,
+                                           norm=dict(eps=1e-5), embedding=dict(scale=1.0)))
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    steps, warmup, batch, context, prompt_len = args.steps or 64, max(args.warmup, 3), args.batch or 8, 1280, 2048
+    common = (dev, flush, steps, warmup, batch, context, prompt_len)
+    r, c = measure_design(xcfg, z["vocab"], *common), measure_design(ccfg, z["vocab"], *common)
+    T = prompt_len
+    keys = T * (T + 1) // 2                                                    # visible (query, key) pairs of a prompt
+    seen = sum(min(t + 1, z["window"]) for t in range(T))
+    row = (z["kv_rank"] + z["lat_rot"] + 15) // 16 * 16                        # the cached row of a latent layer
+    LH, dn, dr, ldv = z["lat_heads"], z["lat_dim"], z["lat_rot"], z["lat_vdim"]
+    tf, gb = pk["bf16_burst"] * 1e12, pk["hbm_gbs"] * 1e9
+    qkv_cols, kv_row = (H + G) * d + G * dv, G * (d + dv) * 2.0
+    dcols, state = 2 * DG * dd + DH * ddv, DH * dd * ddv * 4.0
+    lcols = DH * (2 * dd + ddv)
+    own_lat, c_lat = (z["q_rank"] + z["kv_rank"] + dr + LH), LH * (dn + dr) + z["kv_rank"] + dr + LH * ldv
+    heads = 2 * 2.0 * T * LH * z["kv_rank"] * (dn + ldv)
+    attn = [(k, 2 * 2.0 * H * (d + dv) * keys, "flops") for k in ("attn_headmix_prefill", f"attn_prefill_mma_kernel<{d}")]
+    attn_d = [(k, 2 * batch * context * kv_row, "bytes") for k in ("attn_headmix_decode", f"attn_decode_mma_kernel<{d}")]
+    qkv = ("qkv_finish", 2 * T * (qkv_cols * 6.0 + kv_row), "bytes")
+    rows = [
+        ("papusun prefill", r["prefill_kernels"], attn + [
+            (f"attn_prefill_mma_kernel<{row}", 2 * 2.0 * LH * 2 * row * seen, "flops"),
+            ("fast_kernel<128, 32, 4, true>", heads, "flops"), qkv,
+            ("latent_rows", T * (own_lat * 2 + 2 * LH * (dn + dr) + 2 * z["q_rank"] + 2 * row + 2 * LH * row) * 2.0, "bytes"),
+            ("delta_rows", 2 * T * (dcols * 2 + DH * 4 + DG) * 4.0, "bytes"),
+            ("delta_scan", 2 * T * (dcols + DH * 2 + DG + DH * ddv) * 4.0, "bytes"),
+            ("head_norm_gate", 2 * T * DH * ddv * (4 + 4 + 2.0), "bytes"),
+            ("scaled_sum", 2 * T * W * 3 * 4.0, "bytes"),
+            ("table_gate", 4 * T * z["side"] * (4 + 2 + 2.0), "bytes"),
+            ("layernorm_kernel", (8 * 3.5 * 4.0 - 2 * 3.5 * 4.0 + 6.0) * T * W, "bytes"),
+            ("residual_rmsnorm", 4 * 3.5 * T * W * 4.0, "bytes"),
+            ("gemm_tc2_kernel<1>", 4 * 2.0 * T * W * 2 * ff, "flops"),
+        ]),
+        ("closest prefill", c["prefill_kernels"], attn + [
+            (f"attn_prefill_mma_kernel<{row}", 2 * 2.0 * LH * 2 * row * keys, "flops"),
+            ("fast_kernel<128, 32, 4, true>", heads, "flops"), qkv,
+            ("latent_rows", 2 * T * (LH * dr + z["kv_rank"] + dr + 2 * row + LH * (row - z["kv_rank"])) * 2.0, "bytes"),
+            ("bias_act", 2 * T * (lcols * 2 * 4.0 + ff * 3 // 2 * 6.0 * 2), "bytes"),
+            ("decay_scan", 2 * T * (lcols + DH * ddv) * 4.0, "bytes"),
+            ("norm_sigmoid_gate", 2 * T * (DH * ddv * (4 + 4 + 2.0) + LH * ldv * 6.0), "bytes"),
+            ("residual_rmsnorm", (10 * 3.5 * 4.0) * T * W, "bytes"),
+        ]),
+        ("papusun decode", r["decode_kernels"], attn_d + [
+            (f"attn_decode_mma_kernel<{row}", 2 * batch * min(context, z["window"]) * row * 2.0, "bytes"),
+            ("fast_kernel<64, 64, 4, true>", 2 * LH * z["kv_rank"] * (dn + ldv) * 2.0, "bytes"),
+            ("delta_scan", 2 * batch * state * 2, "bytes"),
+            ("delta_rows", 2 * batch * dcols * (z["conv"] * 2) * 4.0, "bytes"),
+            ("head_norm_gate", 2 * batch * DH * ddv * 10.0, "bytes"),
+            ("skinny", 2.0 * (2 * W * (qkv_cols + H * dv + dcols + 2 * DH + 2 * DH * ddv)
+                              + W * (2 * (z["q_rank"] + LH + LH * ldv) + z["kv_rank"] + dr) + 2 * z["q_rank"] * LH * (dn + dr)
+                              + 4 * W * (3 * ff + 2 * z["side"])), "bytes"),
+        ]),
+        ("closest decode", c["decode_kernels"], attn_d + [
+            (f"attn_decode_mma_kernel<{row}", 2 * batch * context * row * 2.0, "bytes"),
+            ("fast_kernel<64, 64, 4, true>", 2 * LH * z["kv_rank"] * (dn + ldv) * 2.0, "bytes"),
+            ("decay_scan", 2 * batch * state * 2, "bytes"),
+            ("norm_sigmoid_gate", 2 * batch * (DH * ddv * 10.0 + LH * ldv * 6.0), "bytes"),
+            ("skinny", 2.0 * (2 * W * (qkv_cols + H * dv + lcols + 2 * DH * ddv) + 2 * W * (c_lat + LH * ldv) + 4 * W * 3 * ff), "bytes"),
+        ]),
+    ]
+    table = []
+    for title, kern, wanted in rows:
+        for frag, work, bound in wanted:
+            us = sum(v["us"] for k, v in kern.items() if frag in k)
+            n = sum(v["n"] for k, v in kern.items() if frag in k)
+            if not n:
+                continue
+            frac = work / (us * 1e-6) / (tf if bound == "flops" else gb)
+            table.append({"step": title, "kernel": frag, "launches": n, "us": round(us, 2),
+                          "bound": "tensor" if bound == "flops" else "hbm", "frac_of_measured_peak": round(frac, 4)})
+    result = {
+        "metric": f"Papusun decode tokens/s (size {name}, batch {batch}, context {context}) beside Ritirax at equal sizes",
+        "value": round(batch * 1000.0 / r["decode_ms"], 1), "unit": "tokens/s", "n_gpus": 1, "steps": steps,
+        "warmup": warmup, "ms_per_step": round(r["decode_ms"], 4), "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic (random weights, uniform random token ids)",
+        "impl": "brolm_b200", "clocks": r["clocks"], "gpu_launches": r["launches"],
+        "config": {"model": "Papusun", **{k: v for k, v in z.items()}, "layers": len(layers), "global_batch": batch,
+                   "seq_len": context, "closest": {"model": "Ritirax", "layers": [l["type"] for l in clayers]},
+                   "l2": "the prompt is timed after an L2 flush; a decode step reads more than the L2 holds",
+                   "peaks": pk["source"]},
+        "papusun": {"prefill_tok_s": round(T * 1000.0 / r["prefill_ms"], 1), "prefill_ms": round(r["prefill_ms"], 3),
+                    "decode_tok_s": round(batch * 1000.0 / r["decode_ms"], 1), "decode_ms": round(r["decode_ms"], 4)},
+        "closest": {"prefill_tok_s": round(T * 1000.0 / c["prefill_ms"], 1), "prefill_ms": round(c["prefill_ms"], 3),
+                    "decode_tok_s": round(batch * 1000.0 / c["decode_ms"], 1), "decode_ms": round(c["decode_ms"], 4)},
+        "kernels": table,
+        "by_kernel_us": {"papusun_prefill": _top(r["prefill_kernels"], 36), "closest_prefill": _top(c["prefill_kernels"], 36),
+                         "papusun_decode": _top(r["decode_kernels"], 36), "closest_decode": _top(c["decode_kernels"], 36)},
+    }
+    print(json.dumps(result))
+    return 0
+
+
 def _by_kernel(events) -> dict:
     """Device records -> {kernel name: {"us": total time, "n": launches}}."""
     out: dict = {}
@@ -808,9 +948,9 @@ def _top(kern: dict, n: int = 14) -> dict:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--arch", default="gemma2", choices=["gemma2", "banevik", "neburax", "kedasun", "ritirax", "relulix"],
+    ap.add_argument("--arch", default="gemma2", choices=["gemma2", "banevik", "neburax", "kedasun", "ritirax", "relulix", "papusun"],
                     help="banevik, neburax, kedasun: that design at real layer sizes beside Gemma 2 at equal sizes (--size s|m); "
-                         "ritirax: beside Neburax at equal sizes; relulix: beside Ritirax at equal sizes")
+                         "ritirax: beside Neburax at equal sizes; relulix, papusun: beside Ritirax at equal sizes")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=0, help="decode steps in a timed region (default 64; 128 for 9b)")
     ap.add_argument("--warmup", type=int, default=8)
@@ -842,6 +982,8 @@ def main() -> int:
         return ritirax_main(args, peaks())
     if args.arch == "relulix":
         return relulix_main(args, peaks())
+    if args.arch == "papusun":
+        return papusun_main(args, peaks())
     if args.size not in SIZES:
         print(f"bench.py: --size {args.size} goes with --arch banevik, neburax or kedasun")
         return 2

@@ -862,8 +862,9 @@ def papusun_main(args, pk) -> int:
             (f"attn_prefill_mma_kernel<{row}", 2 * 2.0 * LH * 2 * row * seen, "flops"),
             ("fast_kernel<128, 32, 4, true>", heads, "flops"), qkv,
             ("latent_rows", T * (own_lat * 2 + 2 * LH * (dn + dr) + 2 * z["q_rank"] + 2 * row + 2 * LH * row) * 2.0, "bytes"),
-            ("delta_rows", 2 * T * (dcols * 2 + DH * 4 + DG) * 4.0, "bytes"),
-            ("delta_scan", 2 * T * (dcols + DH * 2 + DG + DH * ddv) * 4.0, "bytes"),
+            ("delta_rows", 2 * T * (dcols * 2 + DH * 4) * 4.0, "bytes"),
+            ("delta_chunks", 2 * T * (2 * DG * dd + DH * 46) * 4.0, "bytes"),
+            ("delta_scan", 2 * T * (dcols + DH * 44 + DH * ddv) * 4.0, "bytes"),
             ("head_norm_gate", 2 * T * DH * ddv * (4 + 4 + 2.0), "bytes"),
             ("scaled_sum", 2 * T * W * 3 * 4.0, "bytes"),
             ("table_gate", 4 * T * z["side"] * (4 + 2 + 2.0), "bytes"),
@@ -883,8 +884,7 @@ def papusun_main(args, pk) -> int:
         ("papusun decode", r["decode_kernels"], attn_d + [
             (f"attn_decode_mma_kernel<{row}", 2 * batch * min(context, z["window"]) * row * 2.0, "bytes"),
             ("fast_kernel<64, 64, 4, true>", 2 * LH * z["kv_rank"] * (dn + ldv) * 2.0, "bytes"),
-            ("delta_scan", 2 * batch * state * 2, "bytes"),
-            ("delta_rows", 2 * batch * dcols * (z["conv"] * 2) * 4.0, "bytes"),
+            ("delta_step", 2 * batch * (state * 2 + dcols * (z["conv"] + 1) * 4.0), "bytes"),
             ("head_norm_gate", 2 * batch * DH * ddv * 10.0, "bytes"),
             ("skinny", 2.0 * (2 * W * (qkv_cols + H * dv + dcols + 2 * DH + 2 * DH * ddv)
                               + W * (2 * (z["q_rank"] + LH + LH * ldv) + z["kv_rank"] + dr) + 2 * z["q_rank"] * LH * (dn + dr)

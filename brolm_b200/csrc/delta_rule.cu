@@ -3,25 +3,33 @@
 //
 //     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
 //
-// H value heads of dv entries; G query/key heads of d entries, head h using q/k head h / (H / G).
-//
-// delta_rows makes the recurrence's inputs of a token from its projection row [q: G d | k: G d | v: H dv | zb: H | za: H]:
-//     * a causal convolution over time per channel of q, k and v (K taps, column K - 1 the token's own; the K - 1
-//       inputs before the step come from the rows the state keeps, zeros before the sequence's start), then silu;
+// H value heads of dv entries; G query/key heads of d entries, head h using q/k head h / (H / G).  A token's projection
+// row is [q: G d | k: G d | v: H dv | zb: H | za: H]; its inputs of the recurrence are
+//     * q, k and v after a causal convolution over time per channel (K taps, the last one the token's own; zeros before
+//       the sequence's start) and silu;
 //     * q and k as unit vectors per head, x / sqrt(sum(x^2) + norm_eps); q also times q_scale;
-//     * beta = sigmoid(zb), and g - 1 = expm1(-exp(A_log) softplus(za + dt_bias)): a g close to one keeps in g - 1 the
-//       digits that it loses itself when it is rounded to a float;
-//     * q . k of every q/k head.
-//   In a step of single tokens it also moves the kept inputs on (a prompt leaves that to conv_tail).
+//     * beta = sigmoid(zb), log g = -exp(A_log) softplus(za + dt_bias).
+// The decay is kept as its logarithm and applied as S + expm1(log g) S: a g close to one keeps the digits that it loses
+// itself when it is rounded to a float.
 //
-// delta_scan runs the recurrence.  With o = g S^T q + (q . k) u both sums over d are taken of the state as the token
-// found it, so a token waits for one sum over a column (the one with k), and those with q are folded across the lanes
-// sixteen tokens at once.  The state row of a sequence is laid out [head][value column][d padded to four], read at the
-// start of the sequence's tokens of a step and written at their end; a row b with kv_len[b] <= 0 is padding.
+// A sequence's state row holds S as [head][value column][d padded to four] and, from tail_off on, the convolution's
+// newest inputs as a ring of K rows, position p in row p mod K (no rows for K = 1): a step of single tokens reads K - 1
+// rows and writes the one that no block of the launch reads.  A row b with kv_len[b] <= 0 is padding.
+//
+// A step of single tokens is one kernel, delta_step.  A prompt runs
+//     delta_rows     the inputs of the recurrence, token by token;
+//     delta_tail     the newest inputs into the ring;
+//     delta_chunks   per sixteen tokens and head, what does not hang on the state;
+//     delta_scan     the recurrence, sixteen tokens at a time.
+// With S0 the state ahead of the sixteen tokens, D(i, j) the product of the decays of tokens j + 1 .. i and D(i) that of
+// the tokens up to i, the recurrence's u solve a triangular system whose matrix needs the keys and gates alone:
+//     u_i + sum_{j < i} beta_i D(i, j) (k_i . k_j) u_j = beta_i (v_i - D(i) S0^T k_i) =: r_i,       u = T r
+//     o_i = D(i) S0^T q_i + sum_{j <= i} D(i, j) (q_i . k_j) u_j
+//     S   = D(15) S0 + sum_j D(15, j) k_j u_j^T
+// so all products with S0 of the sixteen tokens are independent of one another.  T's entries are at most one in
+// magnitude (they are entries of products of contractions), every D is the exponential of a sum of its own.
 //
 // Everything is float arithmetic.
-#include <type_traits>
-
 #include "common.cuh"
 
 namespace {
@@ -29,11 +37,28 @@ namespace {
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 
-struct RowsArgs {
+typedef unsigned long long f32x2;          // two floats, for the paired multiply-add
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+
+struct DeltaArgs {
     const float* proj;        // [tokens][ldp]
     long ldp;
     const float* taps;        // [K][C] (tap-major), C = 2 G d + H dv
-    int K, G, d, H, dv;
+    int K, G, d, H, dv, dp;   // dp: d rounded up to a multiple of four
     float norm_eps, q_scale;
     const float* a_log;       // [H]
     const float* dt_bias;     // [H]
@@ -44,19 +69,27 @@ struct RowsArgs {
     const int32_t* slots;
     float* state;
     long state_stride, tail_off;
-    int move_tail;            // every sequence brings one token: the kept inputs are moved on here
     float* u;                 // [tokens][ldu]: q | k | v
     long ldu;
-    float* gates;             // [tokens][2 H]: (g - 1, beta) head by head
-    float* qk;                // [tokens][G]
+    float* gates;             // [tokens][2 H]: (log g, beta) head by head
+    float* chunks;            // [chunk][H][REC]
+    float* out;               // [tokens][ldo]; head h at h * dv
+    long ldo;
+    int tokens, vec;
 };
 
-constexpr int ROWS_WARPS = 8;
-constexpr int V_CHUNK = 128;  // value channels a warp takes at a time
+__device__ __forceinline__ float log_decay(const DeltaArgs& a, float za, int h) {
+    return -expf(a.a_log[h]) * softplus_f(za + a.dt_bias[h]);
+}
 
-// NJ: channels a lane holds of a q or k head (d <= 32 NJ).
-template <int NJ>
-__global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a) {
+// ---------------------------------------------------------------------------
+// delta_rows, any sizes: a warp takes a unit (a q/k head, 128 value channels, or the gates of 32 heads) of a token.
+// ---------------------------------------------------------------------------
+constexpr int ROWS_WARPS = 8;
+constexpr int V_CHUNK = 128;
+
+template <int NJ>             // d <= 32 NJ
+__global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(DeltaArgs a) {
     pdl_trigger();
     const int t = blockIdx.x;
     const int pos = a.positions[t];
@@ -65,11 +98,11 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a)
     const int b = a.tok_seq[t];
     const int q0 = a.cu_q[b], first = a.kv_len[b] - (a.cu_q[b + 1] - q0);
     const int K = a.K, qk_cols = a.G * a.d, v_cols = a.H * a.dv, C = 2 * qk_cols + v_cols;
-    float* tail = a.state + (size_t)a.slots[b] * a.state_stride + a.tail_off;
-    // tap j of channel c reads row_of(j)[c]
-    auto row_of = [&](int j) -> const float* {
+    const float* ring = a.state + (size_t)a.slots[b] * a.state_stride + a.tail_off;
+    const int j0 = max(0, K - 1 - pos);                    // taps ahead of it weigh positions before the start
+    auto row_of = [&](int j) -> const float* {             // tap j of channel c reads row_of(j)[c]
         const int q = pos - (K - 1) + j;
-        return q >= first ? a.proj + (size_t)(q0 + q - first) * a.ldp : tail + (size_t)(q - first + K - 1) * C;
+        return q >= first ? a.proj + (size_t)(q0 + q - first) * a.ldp : ring + (size_t)(q % K) * C;
     };
     float* urow = a.u + (size_t)t * a.ldu;
     const int v_units = (v_cols + V_CHUNK - 1) / V_CHUNK, units = a.G + v_units + (a.H + 31) / 32;
@@ -80,7 +113,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a)
             float q[NJ], k[NJ];
 #pragma unroll
             for (int n = 0; n < NJ; ++n) q[n] = k[n] = 0.0f;
-            for (int j = 0; j < K; ++j) {
+            for (int j = j0; j < K; ++j) {
                 const float* r = row_of(j);
                 const float* w = a.taps + (size_t)j * C;
 #pragma unroll
@@ -92,19 +125,15 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a)
                     }
                 }
             }
-            float sq = 0.0f, sk = 0.0f, dot = 0.0f;
+            float sq = 0.0f, sk = 0.0f;
 #pragma unroll
             for (int n = 0; n < NJ; ++n) {
-                q[n] = silu_f(q[n]);                    // silu(0) = 0: channels beyond d stay zero
+                q[n] = silu_f(q[n]);                        // silu(0) = 0: channels beyond d stay zero
                 k[n] = silu_f(k[n]);
                 sq = fmaf(q[n], q[n], sq);
                 sk = fmaf(k[n], k[n], sk);
-                dot = fmaf(q[n], k[n], dot);
             }
-            sq = warp_sum(sq);
-            sk = warp_sum(sk);
-            dot = warp_sum(dot);
-            const float iq = a.q_scale / sqrtf(sq + a.norm_eps), ik = 1.0f / sqrtf(sk + a.norm_eps);
+            const float iq = a.q_scale / sqrtf(warp_sum(sq) + a.norm_eps), ik = 1.0f / sqrtf(warp_sum(sk) + a.norm_eps);
 #pragma unroll
             for (int n = 0; n < NJ; ++n) {
                 const int c = lane + 32 * n;
@@ -113,24 +142,12 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a)
                     urow[ck + c] = k[n] * ik;
                 }
             }
-            if (lane == 0) a.qk[(size_t)t * a.G + unit] = dot * iq * ik;
-            if (a.move_tail && K > 1) {
-                for (int kk = 0; kk < K - 1; ++kk) {
-                    const float* r = row_of(kk + 1);
-                    float* dst = tail + (size_t)kk * C;
-                    for (int c = lane; c < a.d; c += 32) {
-                        const float x = r[cq + c], y = r[ck + c];
-                        dst[cq + c] = x;
-                        dst[ck + c] = y;
-                    }
-                }
-            }
         } else if (unit < a.G + v_units) {
             const int c0 = 2 * qk_cols + (unit - a.G) * V_CHUNK;
             float v[V_CHUNK / 32];
 #pragma unroll
             for (int n = 0; n < V_CHUNK / 32; ++n) v[n] = 0.0f;
-            for (int j = 0; j < K; ++j) {
+            for (int j = j0; j < K; ++j) {
                 const float* r = row_of(j);
                 const float* w = a.taps + (size_t)j * C;
 #pragma unroll
@@ -144,20 +161,12 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a)
                 const int c = c0 + lane + 32 * n;
                 if (c < C) urow[c] = silu_f(v[n]);
             }
-            if (a.move_tail && K > 1) {
-                for (int kk = 0; kk < K - 1; ++kk) {
-                    const float* r = row_of(kk + 1);
-                    float* dst = tail + (size_t)kk * C;
-                    for (int c = c0 + lane; c < min(c0 + V_CHUNK, C); c += 32) dst[c] = r[c];
-                }
-            }
         } else {
             const int h = (unit - a.G - v_units) * 32 + lane;
             if (h < a.H) {
                 const float* z = a.proj + (size_t)t * a.ldp + C;
-                const float dt = softplus_f(z[a.H + h] + a.dt_bias[h]);
                 float2 g;
-                g.x = expm1f(-expf(a.a_log[h]) * dt);
+                g.x = log_decay(a, z[a.H + h], h);
                 g.y = 1.0f / (1.0f + expf(-z[h]));
                 *reinterpret_cast<float2*>(a.gates + ((size_t)t * a.H + h) * 2) = g;
             }
@@ -165,26 +174,365 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(RowsArgs a)
     }
 }
 
-struct ScanArgs {
-    const float* u;           // [tokens][ld]: q | k | v
-    long ld;
-    const float* gates;       // [tokens][2 H]
-    const float* qk;          // [tokens][G]
-    int G, H, d, dv, dp;      // dp: d rounded up to a multiple of four
-    const int32_t* cu_q;
-    const int32_t* kv_len;
-    const int32_t* slots;
-    float* state;
-    long state_stride;
-    float* out;               // [tokens][ldo]; head h at h * dv
-    long ldo;
-    int ds;                   // lanes per value column (a power of two, at most 32)
-    int vec;                  // every run of q, k and v starts at a multiple of 16 bytes
-    int early;                // a step of single tokens: takes part in programmatic launch
-};
+// The same for up to four taps and sizes in fours: a warp takes its unit of a run of eight packed tokens, four channels
+// a lane and load; the taps' inputs slide through registers, so a token costs one load where the sequence goes on.
+constexpr int RUN = 8, RUN_TAPS = 4;
 
-constexpr int SCAN_TC = 16;
+__device__ __forceinline__ float4 fma4(float4 w, float4 x, float4 c) {
+    return make_float4(fmaf(w.x, x.x, c.x), fmaf(w.y, x.y, c.y), fmaf(w.z, x.z, c.z), fmaf(w.w, x.w, c.w));
+}
+__device__ __forceinline__ float4 silu4(float4 v) { return make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w)); }
+__device__ __forceinline__ float dot4(float4 a, float4 b, float s) {
+    return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s))));
+}
+__device__ __forceinline__ float4 mul4(float4 a, float f) { return make_float4(a.x * f, a.y * f, a.z * f, a.w * f); }
 
+// N columns of four channels a lane (col[n] < 0: none), the convolved and activated values handed to `use` per token.
+template <int N, typename F>
+__device__ __forceinline__ void run_of_tokens(const DeltaArgs& a, int C, const int (&col)[N], F use) {
+    const int K = a.K, t0 = blockIdx.x * RUN;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 w[RUN_TAPS][N], win[RUN_TAPS][N];
+#pragma unroll
+    for (int jj = 0; jj < RUN_TAPS; ++jj)
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            const int j = jj - (RUN_TAPS - K);
+            w[jj][n] = j >= 0 && col[n] >= 0 ? *reinterpret_cast<const float4*>(a.taps + (size_t)j * C + col[n]) : zero;
+            win[jj][n] = zero;
+        }
+    pdl_wait();
+    int prev_b = -1, prev_pos = -2;
+    for (int i = 0; i < RUN && t0 + i < a.tokens; ++i) {
+        const int t = t0 + i, pos = a.positions[t];
+        if (pos < 0) { prev_b = -1; continue; }
+        const int b = a.tok_seq[t];
+        const bool on = b == prev_b && pos == prev_pos + 1;
+        if (on) {
+#pragma unroll
+            for (int jj = 0; jj < RUN_TAPS - 1; ++jj)
+#pragma unroll
+                for (int n = 0; n < N; ++n) win[jj][n] = win[jj + 1][n];
+        } else {
+            const int q0 = a.cu_q[b], first = a.kv_len[b] - (a.cu_q[b + 1] - q0);
+            const float* ring = a.state + (size_t)a.slots[b] * a.state_stride + a.tail_off;
+#pragma unroll
+            for (int jj = 0; jj < RUN_TAPS - 1; ++jj) {
+                const int q = pos - (RUN_TAPS - 1) + jj;
+                const bool in = q >= 0 && jj >= RUN_TAPS - K;
+                const float* r = q >= first ? a.proj + (size_t)(q0 + q - first) * a.ldp : ring + (size_t)(in ? q % K : 0) * C;
+#pragma unroll
+                for (int n = 0; n < N; ++n) win[jj][n] = in && col[n] >= 0 ? *reinterpret_cast<const float4*>(r + col[n]) : zero;
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < N; ++n)
+            win[RUN_TAPS - 1][n] = col[n] >= 0 ? *reinterpret_cast<const float4*>(a.proj + (size_t)t * a.ldp + col[n]) : zero;
+        prev_b = b;
+        prev_pos = pos;
+        float4 v[N];
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+            v[n] = zero;
+#pragma unroll
+            for (int jj = 0; jj < RUN_TAPS; ++jj) v[n] = fma4(w[jj][n], win[jj][n], v[n]);
+            v[n] = silu4(v[n]);
+        }
+        use(t, v);
+    }
+}
+
+template <int NV>             // d <= 128 NV
+__global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_run_kernel(DeltaArgs a) {
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int qk_cols = a.G * a.d, v_cols = a.H * a.dv, C = 2 * qk_cols + v_cols;
+    const int v_units = (v_cols + V_CHUNK - 1) / V_CHUNK, units = a.G + v_units + 1;
+    const int unit = blockIdx.y * ROWS_WARPS + warp;
+    if (unit >= units) return;
+    if (unit < a.G) {
+        int col[2 * NV];
+#pragma unroll
+        for (int n = 0; n < NV; ++n) {
+            const int c = lane * 4 + 128 * n;
+            col[n] = c < a.d ? unit * a.d + c : -1;
+            col[NV + n] = c < a.d ? qk_cols + unit * a.d + c : -1;
+        }
+        run_of_tokens<2 * NV>(a, C, col, [&](int t, const float4 (&v)[2 * NV]) {
+            float sq = 0.0f, sk = 0.0f;
+#pragma unroll
+            for (int n = 0; n < NV; ++n) {
+                sq = dot4(v[n], v[n], sq);
+                sk = dot4(v[NV + n], v[NV + n], sk);
+            }
+            const float iq = a.q_scale / sqrtf(warp_sum(sq) + a.norm_eps), ik = 1.0f / sqrtf(warp_sum(sk) + a.norm_eps);
+            float* urow = a.u + (size_t)t * a.ldu;
+#pragma unroll
+            for (int n = 0; n < NV; ++n)
+                if (col[n] >= 0) {
+                    *reinterpret_cast<float4*>(urow + col[n]) = mul4(v[n], iq);
+                    *reinterpret_cast<float4*>(urow + col[NV + n]) = mul4(v[NV + n], ik);
+                }
+        });
+    } else if (unit < a.G + v_units) {
+        const int c = 2 * qk_cols + (unit - a.G) * V_CHUNK + lane * 4;
+        const int col[1] = {c < C ? c : -1};
+        run_of_tokens<1>(a, C, col, [&](int t, const float4 (&v)[1]) {
+            if (col[0] >= 0) *reinterpret_cast<float4*>(a.u + (size_t)t * a.ldu + col[0]) = v[0];
+        });
+    } else {
+        pdl_wait();
+        const int t0 = blockIdx.x * RUN, n = min(RUN, a.tokens - t0) * a.H;
+        for (int i = lane; i < n; i += 32) {
+            const int t = t0 + i / a.H, h = i % a.H;
+            if (a.positions[t] < 0) continue;
+            const float* z = a.proj + (size_t)t * a.ldp + C;
+            float2 g;
+            g.x = log_decay(a, z[a.H + h], h);
+            g.y = 1.0f / (1.0f + expf(-z[h]));
+            *reinterpret_cast<float2*>(a.gates + ((size_t)t * a.H + h) * 2) = g;
+        }
+    }
+}
+
+// ring[p mod K][c] <- the input of position p, for the newest K - 1 positions of every sequence (after all that read it).
+__global__ void __launch_bounds__(256) delta_tail_kernel(DeltaArgs a) {
+    pdl_trigger();
+    const int b = blockIdx.x, C = 2 * a.G * a.d + a.H * a.dv;
+    const int c = blockIdx.y * blockDim.x + threadIdx.x;
+    const int kv_len = a.kv_len[b];
+    if (kv_len <= 0 || c >= C) return;
+    const int q0 = a.cu_q[b], first = kv_len - (a.cu_q[b + 1] - q0);
+    float* ring = a.state + (size_t)a.slots[b] * a.state_stride + a.tail_off;
+    pdl_wait();
+    for (int p = max(first, kv_len - (a.K - 1)); p < kv_len; ++p)
+        ring[(size_t)(p % a.K) * C + c] = a.proj[(size_t)(q0 + p - first) * a.ldp + c];
+}
+
+// ---------------------------------------------------------------------------
+// A step of single tokens: convolution, unit norms, gates and the recurrence.  A block of 128 threads takes one
+// (sequence, head) and 128 / DS value columns; the DS lanes of a column keep NJ float4 of its states each (entries
+// 4 (j DS + ds) + e).  Every block of a head makes the head's q and k (a channel or a few per thread).
+// ---------------------------------------------------------------------------
+template <int NJ, int DS>
+__global__ void __launch_bounds__(128) delta_step_kernel(DeltaArgs a) {
+    constexpr int DP = 4 * NJ * DS, VT = 128 / DS, CH = (DP + 127) / 128;
+    __shared__ __align__(16) float sq[DP], sk[DP];
+    __shared__ float sv[VT], red[3][4];
+    pdl_trigger();
+    const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VT;
+    const int kv_len = a.kv_len[b];
+    if (kv_len <= 0) return;
+    const int t = a.cu_q[b], pos = kv_len - 1, K = a.K;
+    const int share = a.H / a.G, hk = h / share;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int ds = tid % DS, vcol = tid / DS, v = v0 + vcol;
+    const bool live = v < a.dv;
+    const int dp4 = a.dp >> 2, qk_cols = a.G * a.d, C = 2 * qk_cols + a.H * a.dv;
+    float* row = a.state + (size_t)a.slots[b] * a.state_stride;
+    float* st = row + ((size_t)h * a.dv + (live ? v : 0)) * a.dp;
+    float* ring = row + a.tail_off;
+    // The state and the kept inputs were written by the step before: they are fetched, and the convolution's older taps
+    // summed, while the product ahead of this kernel finishes.
+    float4 S[NJ];
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        const int f = j * DS + ds;
+        S[j] = live && f < dp4 ? *reinterpret_cast<const float4*>(st + 4 * f) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+    float aq[CH], ak[CH], av = 0.0f;
+#pragma unroll
+    for (int n = 0; n < CH; ++n) aq[n] = ak[n] = 0.0f;
+    const int cq = hk * a.d, ck = qk_cols + hk * a.d, cv = 2 * qk_cols + h * a.dv + v0 + tid;
+    const bool own_v = tid < VT && v0 + tid < a.dv;
+    for (int j = max(0, K - 1 - pos); j < K - 1; ++j) {
+        const float* r = ring + (size_t)((pos - (K - 1) + j) % K) * C;
+        const float* w = a.taps + (size_t)j * C;
+#pragma unroll
+        for (int n = 0; n < CH; ++n) {
+            const int c = tid + 128 * n;
+            if (c < a.d) {
+                aq[n] = fmaf(w[cq + c], r[cq + c], aq[n]);
+                ak[n] = fmaf(w[ck + c], r[ck + c], ak[n]);
+            }
+        }
+        if (own_v) av = fmaf(w[cv], r[cv], av);
+    }
+    const float* w = a.taps + (size_t)(K - 1) * C;
+    float wq[CH], wk[CH];
+#pragma unroll
+    for (int n = 0; n < CH; ++n) {
+        const int c = tid + 128 * n;
+        wq[n] = c < a.d ? w[cq + c] : 0.0f;
+        wk[n] = c < a.d ? w[ck + c] : 0.0f;
+    }
+    const float wv = own_v ? w[cv] : 0.0f, neg_a = -expf(a.a_log[h]), dtb = a.dt_bias[h];
+    pdl_wait();
+    const float* x = a.proj + (size_t)t * a.ldp;
+    float* keep = ring + (size_t)(pos % K) * C;
+    const bool keeps_qk = K > 1 && blockIdx.x == 0 && h == hk * share;
+    const float zb = x[C + h], za = x[C + a.H + h];
+    float s0 = 0.0f, s1 = 0.0f, s2 = 0.0f;
+#pragma unroll
+    for (int n = 0; n < CH; ++n) {
+        const int c = tid + 128 * n;
+        if (c < a.d) {
+            const float xq = x[cq + c], xk = x[ck + c];
+            const float q = silu_f(fmaf(wq[n], xq, aq[n])), k = silu_f(fmaf(wk[n], xk, ak[n]));
+            sq[c] = q;
+            sk[c] = k;
+            s0 = fmaf(q, q, s0);
+            s1 = fmaf(k, k, s1);
+            s2 = fmaf(q, k, s2);
+            if (keeps_qk) { keep[cq + c] = xq; keep[ck + c] = xk; }
+        } else if (c < DP) {
+            sq[c] = sk[c] = 0.0f;
+        }
+    }
+    if (own_v) {
+        const float xv = x[cv];
+        sv[tid] = silu_f(fmaf(wv, xv, av));
+        if (K > 1) keep[cv] = xv;
+    }
+    s0 = warp_sum(s0);
+    s1 = warp_sum(s1);
+    s2 = warp_sum(s2);
+    if (lane == 0) { red[0][warp] = s0; red[1][warp] = s1; red[2][warp] = s2; }
+    const float gm1 = expm1f(neg_a * softplus_f(za + dtb)), beta = 1.0f / (1.0f + expf(-zb));
+    __syncthreads();
+    const float iq = a.q_scale / sqrtf((red[0][0] + red[0][1]) + (red[0][2] + red[0][3]) + a.norm_eps);
+    const float ik = 1.0f / sqrtf((red[1][0] + red[1][1]) + (red[1][2] + red[1][3]) + a.norm_eps);
+    const float qk = ((red[2][0] + red[2][1]) + (red[2][2] + red[2][3])) * iq * ik;
+    float held = 0.0f, read = 0.0f;                        // S^T k and S^T q of the column, before the decay
+    float4 kk[NJ];
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+        kk[j] = reinterpret_cast<const float4*>(sk)[j * DS + ds];
+        const float4 qq = reinterpret_cast<const float4*>(sq)[j * DS + ds];
+        held = dot4(S[j], kk[j], held);
+        read = dot4(S[j], qq, read);
+    }
+#pragma unroll
+    for (int o = DS >> 1; o > 0; o >>= 1) {
+        held += __shfl_xor_sync(0xffffffffu, held, o);
+        read += __shfl_xor_sync(0xffffffffu, read, o);
+    }
+    held *= ik;
+    read *= iq;
+    const float u = beta * ((live ? sv[vcol] : 0.0f) - fmaf(gm1, held, held)), ku = ik * u;
+    if (live) {
+        if (ds == 0) a.out[(size_t)t * a.ldo + (size_t)h * a.dv + v] = fmaf(qk, u, fmaf(gm1, read, read));
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+            const int f = j * DS + ds;
+            if (f < dp4) {
+                S[j].x = fmaf(kk[j].x, ku, fmaf(gm1, S[j].x, S[j].x));
+                S[j].y = fmaf(kk[j].y, ku, fmaf(gm1, S[j].y, S[j].y));
+                S[j].z = fmaf(kk[j].z, ku, fmaf(gm1, S[j].z, S[j].z));
+                S[j].w = fmaf(kk[j].w, ku, fmaf(gm1, S[j].w, S[j].w));
+                *reinterpret_cast<float4*>(st + 4 * f) = S[j];
+            }
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------
+// delta_chunks: a block takes sixteen tokens of one (sequence, head) and leaves a record of REC floats:
+//   T [16][20], B [16][20] (rows padded against bank conflicts), B_ij = D(i, j) (q_i . k_j) for j <= i,
+//   beta [16], beta_i D(i) [16], D(i) [16], D(15, i) [16], expm1(log D(15)), three unused.
+// Tokens beyond the sequence's end have k = q = 0, log g = 0 and beta = 0, and change nothing.
+// Record number of chunk c of sequence b: cu_q[b] / 16 + b + c (sequences never share one).
+// ---------------------------------------------------------------------------
+constexpr int TC = 16, MR = 20, OFF_B = TC * MR, OFF_V = 2 * TC * MR, REC = OFF_V + 4 * TC + 4;
+
+__device__ __forceinline__ int record_of(int q0, int b, int chunk) { return q0 / TC + b + chunk; }
+
+__global__ void __launch_bounds__(128) delta_chunks_kernel(DeltaArgs a) {
+    extern __shared__ __align__(16) float sm[];            // k [16][ld], q [16][ld]
+    __shared__ float lg[TC], be[TC], A[TC][TC + 1];
+    const int chunk = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
+    const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0, t0 = chunk * TC;
+    if (a.kv_len[b] <= 0 || t0 >= q_len) return;
+    const int n_tok = min(TC, q_len - t0), hk = h / (a.H / a.G), ld = a.dp + 4, dp4 = a.dp >> 2;
+    float* sk = sm;
+    float* sq = sm + TC * ld;
+    float* rec = a.chunks + ((size_t)record_of(q0, b, chunk) * a.H + h) * REC;
+    if (a.vec) {
+        for (int i = tid; i < TC * dp4; i += 128) {
+            const int r = i / dp4, c = (i - r * dp4) * 4;
+            float4 k = make_float4(0.0f, 0.0f, 0.0f, 0.0f), q = k;
+            if (r < n_tok) {
+                const float* row = a.u + (size_t)(q0 + t0 + r) * a.ldu + hk * a.d + c;
+                q = *reinterpret_cast<const float4*>(row);
+                k = *reinterpret_cast<const float4*>(row + a.G * a.d);
+            }
+            *reinterpret_cast<float4*>(sk + r * ld + c) = k;
+            *reinterpret_cast<float4*>(sq + r * ld + c) = q;
+        }
+    } else {
+        for (int i = tid; i < TC * a.dp; i += 128) {
+            const int r = i / a.dp, c = i - r * a.dp;
+            const bool in = r < n_tok && c < a.d;
+            const float* row = a.u + (size_t)(q0 + t0 + (in ? r : 0)) * a.ldu + hk * a.d + (in ? c : 0);
+            sk[r * ld + c] = in ? row[a.G * a.d] : 0.0f;
+            sq[r * ld + c] = in ? row[0] : 0.0f;
+        }
+    }
+    if (tid < TC) {
+        const float2 g = tid < n_tok ? *reinterpret_cast<const float2*>(a.gates + ((size_t)(q0 + t0 + tid) * a.H + h) * 2)
+                                     : make_float2(0.0f, 0.0f);
+        lg[tid] = g.x;
+        be[tid] = g.y;
+    }
+    __syncthreads();
+    // thread (i, jj): the products of row i with rows jj and jj + 8
+    const int i = tid >> 3, jj = tid & 7;
+    float kk[2] = {0.0f, 0.0f}, qk[2] = {0.0f, 0.0f};
+    for (int f = 0; f < dp4; ++f) {
+        const float4 ki = *reinterpret_cast<const float4*>(sk + i * ld + 4 * f), qi = *reinterpret_cast<const float4*>(sq + i * ld + 4 * f);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+            const float4 kj = *reinterpret_cast<const float4*>(sk + (jj + 8 * m) * ld + 4 * f);
+            kk[m] = dot4(ki, kj, kk[m]);
+            qk[m] = dot4(qi, kj, qk[m]);
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+        const int j = jj + 8 * m;
+        float s = 0.0f;
+        for (int l = j + 1; l <= i; ++l) s += lg[l];
+        const float D = i >= j ? expf(s) : 0.0f;
+        A[i][j] = i > j ? be[i] * D * kk[m] : 0.0f;
+        rec[OFF_B + i * MR + j] = D * qk[m];
+        if (i == TC - 1) rec[OFF_V + 3 * TC + j] = D;
+        if (j == 0) {
+            const float s_all = s + lg[0], all = expf(s_all);
+            rec[OFF_V + i] = be[i];
+            rec[OFF_V + TC + i] = be[i] * all;
+            rec[OFF_V + 2 * TC + i] = all;
+            if (i == TC - 1) rec[OFF_V + 4 * TC] = expm1f(s_all);
+        }
+    }
+    __syncthreads();
+    if (tid < TC) {                                        // column tid of T, from the diagonal down
+        float x[TC];
+#pragma unroll
+        for (int r = 0; r < TC; ++r) {
+            float s = 0.0f;
+#pragma unroll
+            for (int j = 0; j < r; ++j) s = fmaf(A[r][j], x[j], s);
+            x[r] = r < tid ? 0.0f : r == tid ? 1.0f : -s;
+        }
+#pragma unroll
+        for (int r = 0; r < TC; ++r) rec[r * MR + tid] = x[r];
+    }
+}
+
+// ---------------------------------------------------------------------------
+// delta_scan: blocks and lanes as in delta_step; sixteen tokens and their record at a time, three stages of cp.async.
+// A warp works on its own columns alone.  Of a column's sixteen sums lane ds ends up with those of tokens ds, ds + DS, ..
+// ---------------------------------------------------------------------------
 __device__ __forceinline__ void cp4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
@@ -192,274 +540,313 @@ __device__ __forceinline__ void cp16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// A block of 128 threads takes one (sequence, head) and 128 / DS value columns; the DS lanes of a column keep NJ float4
-// of the column's states each (entries 4 (j DS + ds) + e).  Tokens are staged sixteen at a time through two buffers.
-// DSC > 0: lanes per column known to the compiler and NJ * DSC float4 are exactly a row of d; DSC = 0: any d.
-template <int NJ, int DSC>
-__global__ void __launch_bounds__(128) delta_scan_kernel(ScanArgs a) {
+constexpr int STAGES = 3, XR = 20;                         // XR: floats between two columns' sixteen exchanged numbers
+
+template <int NJ, int DS> __host__ __device__ constexpr int scan_stage() { return TC * (2 * 4 * NJ * DS + 128 / DS) + REC; }
+template <int NJ, int DS> __host__ __device__ constexpr int scan_floats() { return STAGES * scan_stage<NJ, DS>() + 2 * (128 / DS) * XR; }
+
+template <int NJ, int DS>
+__global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
     extern __shared__ __align__(16) float sm[];
-    if (a.early) pdl_trigger();
-    constexpr bool EXACT = DSC > 0;
-    const int DS = EXACT ? DSC : a.ds, VT = 128 / DS;
-    const int dp = EXACT ? 4 * NJ * DSC : a.dp, dp4 = dp >> 2;
-    const int stage = SCAN_TC * (2 * dp + VT + 4);    // q [TC][dp], k [TC][dp], v [TC][VT], (g - 1, beta, q.k, -) [TC]
+    constexpr int DP = 4 * NJ * DS, VT = 128 / DS, NT = TC / DS, STAGE = scan_stage<NJ, DS>();
     const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VT;
     const int kv_len = a.kv_len[b];
     if (kv_len <= 0) return;
     const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0;
     if (q_len <= 0) return;
-    const int hk = h / (a.H / a.G);
-    const int ds = threadIdx.x % DS, vcol = threadIdx.x / DS, v = v0 + vcol;
+    const int hk = h / (a.H / a.G), tid = threadIdx.x;
+    const int ds = tid % DS, vcol = tid / DS, v = v0 + vcol;
     const bool live = v < a.dv;
-    float* st = a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + (live ? v : 0)) * dp;
-    float S[NJ * 4];
-    // the state is this kernel's own: nothing that runs just before it in the step writes it
+    const int dp4 = a.dp >> 2;
+    float* st = a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + (live ? v : 0)) * a.dp;
+    float* xr = sm + STAGES * STAGE + vcol * XR;           // the column's exchanged r, then u
+    float* xu = xr + VT * XR;
+    f32x2 S[2 * NJ];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
         const int f = j * DS + ds;
         float4 s4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (live && f < dp4) s4 = *reinterpret_cast<const float4*>(st + 4 * f);
-        S[4 * j] = s4.x; S[4 * j + 1] = s4.y; S[4 * j + 2] = s4.z; S[4 * j + 3] = s4.w;
+        S[2 * j] = pack2(s4.x, s4.y);
+        S[2 * j + 1] = pack2(s4.z, s4.w);
     }
-    // the padding of d to a multiple of four, and value columns beyond dv, stay zero in both buffers
-    for (int i = threadIdx.x; i < 2 * stage; i += 128) sm[i] = 0.0f;
-    __syncthreads();
-    pdl_wait();
-    const int n_chunks = (q_len + SCAN_TC - 1) / SCAN_TC;
-    const int vt_here = min(VT, a.dv - v0);
+    const int n_chunks = (q_len + TC - 1) / TC, vt_here = min(VT, a.dv - v0);
+    // rows padded to DP, value columns beyond dv and tokens beyond the end read as zeros
+    if (DP != a.d || vt_here != VT || (q_len & (TC - 1))) {
+        for (int i = tid; i < STAGES * STAGE; i += 128) sm[i] = 0.0f;
+        __syncthreads();
+    }
     const int q_off = hk * a.d, k_off = a.G * a.d + hk * a.d, v_off = 2 * a.G * a.d + h * a.dv + v0;
-
     auto issue = [&](int chunk) {
-        float* sq = sm + (chunk & 1) * stage;
-        float* sk = sq + SCAN_TC * dp;
-        float* sv = sk + SCAN_TC * dp;
-        float* sg = sv + SCAN_TC * VT;
-        const int t0 = chunk * SCAN_TC, n_tok = min(SCAN_TC, q_len - t0);
+        float* sk = sm + (chunk % STAGES) * STAGE;
+        float* sq = sk + TC * DP;
+        float* sv = sq + TC * DP;
+        float* sr = sv + TC * VT;
+        const int t0 = chunk * TC, n_tok = min(TC, q_len - t0);
+        if (n_tok < TC && chunk >= STAGES) {               // the last stage holds older tokens where there are none now
+            for (int i = tid; i < (TC - n_tok) * DP; i += 128) sk[n_tok * DP + i] = sq[n_tok * DP + i] = 0.0f;
+            for (int i = tid; i < (TC - n_tok) * VT; i += 128) sv[n_tok * VT + i] = 0.0f;
+        }
         if (a.vec) {
             const int d4 = a.d >> 2, v4 = vt_here >> 2;
-            for (int idx = threadIdx.x; idx < n_tok * d4; idx += 128) {
+            for (int idx = tid; idx < n_tok * d4; idx += 128) {
                 const int tt = idx / d4, c = (idx - tt * d4) << 2;
-                const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ld + c;
-                cp16(sq + tt * dp + c, row + q_off);
-                cp16(sk + tt * dp + c, row + k_off);
+                const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ldu + c;
+                cp16(sq + tt * DP + c, row + q_off);
+                cp16(sk + tt * DP + c, row + k_off);
             }
-            for (int idx = threadIdx.x; idx < n_tok * v4; idx += 128) {
+            for (int idx = tid; idx < n_tok * v4; idx += 128) {
                 const int tt = idx / v4, c = (idx - tt * v4) << 2;
-                cp16(sv + tt * VT + c, a.u + (size_t)(q0 + t0 + tt) * a.ld + v_off + c);
+                cp16(sv + tt * VT + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
             }
         } else {
-            for (int idx = threadIdx.x; idx < n_tok * a.d; idx += 128) {
+            for (int idx = tid; idx < n_tok * a.d; idx += 128) {
                 const int tt = idx / a.d, c = idx - tt * a.d;
-                const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ld + c;
-                cp4(sq + tt * dp + c, row + q_off);
-                cp4(sk + tt * dp + c, row + k_off);
+                const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ldu + c;
+                cp4(sq + tt * DP + c, row + q_off);
+                cp4(sk + tt * DP + c, row + k_off);
             }
-            for (int idx = threadIdx.x; idx < n_tok * vt_here; idx += 128) {
+            for (int idx = tid; idx < n_tok * vt_here; idx += 128) {
                 const int tt = idx / vt_here, c = idx - tt * vt_here;
-                cp4(sv + tt * VT + c, a.u + (size_t)(q0 + t0 + tt) * a.ld + v_off + c);
+                cp4(sv + tt * VT + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
             }
         }
-        for (int idx = threadIdx.x; idx < n_tok * 3; idx += 128) {
-            const int tt = idx / 3, c = idx - tt * 3;
-            const size_t t = (size_t)(q0 + t0 + tt);
-            cp4(sg + tt * 4 + c, c < 2 ? a.gates + (t * a.H + h) * 2 + c : a.qk + t * a.G + hk);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+        const float* rec = a.chunks + ((size_t)record_of(q0, b, chunk) * a.H + h) * REC;
+        for (int idx = tid; idx < REC / 4; idx += 128) cp16(sr + 4 * idx, rec + 4 * idx);
     };
-
-    issue(0);
+#pragma unroll
+    for (int s = 0; s < STAGES - 1; ++s) {
+        if (s < n_chunks) issue(s);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
     for (int kc = 0; kc < n_chunks; ++kc) {
-        const int t0 = kc * SCAN_TC, n_tok = min(SCAN_TC, q_len - t0);
-        float* sq = sm + (kc & 1) * stage;
-        float* sk = sq + SCAN_TC * dp;
-        float* sv = sk + SCAN_TC * dp;
-        const float4* sg = reinterpret_cast<const float4*>(sv + SCAN_TC * VT);
-        if (kc + 1 < n_chunks) {
-            issue(kc + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        float pv[SCAN_TC];                             // a lane's part of every token's result
-        const float4* q4 = reinterpret_cast<const float4*>(sq) + ds;
-        const float4* k4 = reinterpret_cast<const float4*>(sk) + ds;
-        auto tokens = [&](auto full) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+        __syncthreads();                                   // this stage has landed, and no warp works on the one before
+        if (kc + STAGES - 1 < n_chunks) issue(kc + STAGES - 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        const float* sk = sm + (kc % STAGES) * STAGE;
+        const float* sq = sk + TC * DP;
+        const float* sv = sq + TC * DP;
+        const float* sr = sv + TC * VT;
+        // sixteen sums over the column's d, folded across its lanes: at every step a lane hands half of what it holds to
+        // the lane `o` away and adds what it gets to the half it keeps; p is the token ds + DS (p mod NT) of lane p / NT
+        auto sums = [&](const float* rows, float (&mine)[NT]) {
+            float s[TC];
 #pragma unroll
-            for (int tt = 0; tt < SCAN_TC; ++tt) {
-                pv[tt] = 0.0f;
-                if (decltype(full)::value || tt < n_tok) {
-                    const float vv = sv[tt * VT + vcol];
-                    const float4 g = sg[tt];
-                    float4 kk[NJ];
-                    float kx = 0.0f, ky = 0.0f, kz = 0.0f, kw = 0.0f, qx = 0.0f, qy = 0.0f, qz = 0.0f, qw = 0.0f;
+            for (int p = 0; p < TC; ++p) {
+                const int tok = p / NT + DS * (p % NT);
+                const ulonglong2* r = reinterpret_cast<const ulonglong2*>(rows + tok * DP) + ds;
+                f32x2 acc = 0ull, acc1 = 0ull;
 #pragma unroll
-                    for (int j = 0; j < NJ; ++j) {
-                        if (EXACT || j * DS + ds < dp4) {
-                            const float4 qq = q4[tt * dp4 + j * DS];
-                            kk[j] = k4[tt * dp4 + j * DS];
-                            kx = fmaf(S[4 * j], kk[j].x, kx);
-                            ky = fmaf(S[4 * j + 1], kk[j].y, ky);
-                            kz = fmaf(S[4 * j + 2], kk[j].z, kz);
-                            kw = fmaf(S[4 * j + 3], kk[j].w, kw);
-                            qx = fmaf(S[4 * j], qq.x, qx);
-                            qy = fmaf(S[4 * j + 1], qq.y, qy);
-                            qz = fmaf(S[4 * j + 2], qq.z, qz);
-                            qw = fmaf(S[4 * j + 3], qq.w, qw);
-                        } else {
-                            kk[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                        }
-                    }
-                    float held = (kx + ky) + (kz + kw);                // what the column holds for k, summed over its lanes
-#pragma unroll
-                    for (int o = (EXACT ? DSC : 32) >> 1; o > 0; o >>= 1)
-                        if (EXACT || o < DS) held += __shfl_xor_sync(0xffffffffu, held, o);
-                    const float u = g.y * (vv - fmaf(g.x, held, held));
-                    const float part = (qx + qy) + (qz + qw);
-                    pv[tt] = fmaf(g.x, part, part) + (ds == 0 ? g.z * u : 0.0f);
-#pragma unroll
-                    for (int j = 0; j < NJ; ++j) {
-                        S[4 * j] = fmaf(kk[j].x, u, fmaf(g.x, S[4 * j], S[4 * j]));
-                        S[4 * j + 1] = fmaf(kk[j].y, u, fmaf(g.x, S[4 * j + 1], S[4 * j + 1]));
-                        S[4 * j + 2] = fmaf(kk[j].z, u, fmaf(g.x, S[4 * j + 2], S[4 * j + 2]));
-                        S[4 * j + 3] = fmaf(kk[j].w, u, fmaf(g.x, S[4 * j + 3], S[4 * j + 3]));
-                    }
+                for (int j = 0; j < NJ; ++j) {
+                    const ulonglong2 x = r[j * DS];
+                    acc = fma2(S[2 * j], x.x, acc);
+                    acc1 = fma2(S[2 * j + 1], x.y, acc1);
                 }
+                const float2 e = unpack2(acc), f = unpack2(acc1);
+                s[p] = (e.x + e.y) + (f.x + f.y);
             }
-        };
-        if (n_tok == SCAN_TC) tokens(std::true_type{});
-        else tokens(std::false_type{});
-        if (n_tok == 1) {                              // a single token: its sum alone crosses the lanes
-            float acc = pv[0];
-            for (int o = DS >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-            if (ds == 0 && live) a.out[(size_t)(q0 + t0) * a.ldo + (size_t)h * a.dv + v] = acc;
-            __syncthreads();
-            continue;
-        }
-        // The sixteen sums over a column's DS lanes, all at once: at every step a lane hands half of what it holds to
-        // the lane `o` away and adds what it gets to the half it keeps.  `first` is the first token a lane ends up with.
-        int first = 0, kept = SCAN_TC, o = DS >> 1;
-#define BROLM_FOLD(N)                                                              \
-        if (o > 0) {                                                               \
-            const bool up = (ds & o) != 0;                                         \
-            _Pragma("unroll") for (int i = 0; i < N; ++i) {                        \
-                const float send = up ? pv[i] : pv[i + N];                         \
-                const float keep = up ? pv[i + N] : pv[i];                         \
-                pv[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);              \
-            }                                                                      \
-            if (up) first += N;                                                    \
-            kept = N;                                                              \
-            o >>= 1;                                                               \
-        }
-        BROLM_FOLD(8)
-        BROLM_FOLD(4)
-        BROLM_FOLD(2)
-        BROLM_FOLD(1)
-#undef BROLM_FOLD
-        bool writer = live;
-        if (o > 0) {                                   // 32 lanes a column: two lanes hold halves of one token's sum
-            pv[0] += __shfl_xor_sync(0xffffffffu, pv[0], o);
-            writer = writer && (ds & 1) == 0;
-        }
-        float* orow = a.out + (size_t)(q0 + t0 + first) * a.ldo + (size_t)h * a.dv + v;
 #pragma unroll
-        for (int i = 0; i < SCAN_TC; ++i)
-            if (writer && i < kept && first + i < n_tok) orow[(size_t)i * a.ldo] = pv[i];
-        __syncthreads();                               // the buffer is free for the chunk after the next
+            for (int n = TC / 2, o = DS / 2; o > 0; n >>= 1, o >>= 1) {
+                const bool up = (ds & o) != 0;
+#pragma unroll
+                for (int i = 0; i < TC / 2; ++i)
+                    if (i < n) {
+                        const float send = up ? s[i] : s[i + n], keep = up ? s[i + n] : s[i];
+                        s[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                    }
+            }
+#pragma unroll
+            for (int i = 0; i < NT; ++i) mine[i] = s[i];
+        };
+        float pk[NT], pq[NT];
+        sums(sk, pk);
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+            const int tok = ds + DS * i;
+            xr[tok] = fmaf(-sr[OFF_V + TC + tok], pk[i], sr[OFF_V + tok] * sv[tok * VT + vcol]);
+        }
+        sums(sq, pq);
+        __syncwarp();
+        float u[TC];
+#pragma unroll
+        for (int j = 0; j < TC; j += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(xr + j);
+            u[j] = x.x; u[j + 1] = x.y; u[j + 2] = x.z; u[j + 3] = x.w;
+        }
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+            const int tok = ds + DS * i;
+            float s = 0.0f, s1 = 0.0f;
+#pragma unroll
+            for (int j = 0; j < TC; j += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(sr + tok * MR + j);
+                s = fmaf(m.x, u[j], fmaf(m.y, u[j + 1], s));
+                s1 = fmaf(m.z, u[j + 2], fmaf(m.w, u[j + 3], s1));
+            }
+            xu[tok] = s + s1;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < TC; j += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(xu + j);
+            u[j] = x.x; u[j + 1] = x.y; u[j + 2] = x.z; u[j + 3] = x.w;
+        }
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+            const int tok = ds + DS * i, t = kc * TC + tok;
+            float s = sr[OFF_V + 2 * TC + tok] * pq[i], s1 = 0.0f;
+#pragma unroll
+            for (int j = 0; j < TC; j += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(sr + OFF_B + tok * MR + j);
+                s = fmaf(m.x, u[j], fmaf(m.y, u[j + 1], s));
+                s1 = fmaf(m.z, u[j + 2], fmaf(m.w, u[j + 3], s1));
+            }
+            if (live && t < q_len) a.out[(size_t)(q0 + t) * a.ldo + (size_t)h * a.dv + v] = s + s1;
+        }
+        const float dm1 = sr[OFF_V + 4 * TC];
+        const f32x2 dm2 = pack2(dm1, dm1);
+#pragma unroll
+        for (int j = 0; j < 2 * NJ; ++j) S[j] = fma2(dm2, S[j], S[j]);
+#pragma unroll
+        for (int tok = 0; tok < TC; ++tok) {
+            const float f = sr[OFF_V + 3 * TC + tok] * u[tok];
+            const f32x2 f2 = pack2(f, f);
+            const ulonglong2* r = reinterpret_cast<const ulonglong2*>(sk + tok * DP) + ds;
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+                const ulonglong2 x = r[j * DS];
+                S[2 * j] = fma2(x.x, f2, S[2 * j]);
+                S[2 * j + 1] = fma2(x.y, f2, S[2 * j + 1]);
+            }
+        }
     }
     if (live) {
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
             const int f = j * DS + ds;
-            if (f < dp4) *reinterpret_cast<float4*>(st + 4 * f) = make_float4(S[4 * j], S[4 * j + 1], S[4 * j + 2], S[4 * j + 3]);
+            const float2 e = unpack2(S[2 * j]), g = unpack2(S[2 * j + 1]);
+            if (f < dp4) *reinterpret_cast<float4*>(st + 4 * f) = make_float4(e.x, e.y, g.x, g.y);
         }
     }
 }
 
-template <int NJ, int DSC>
-int launch_scan_as(const ScanArgs& a, dim3 grid, size_t smem, cudaStream_t stream) {
-    static size_t allowed = 0;
-    if (smem > 48 * 1024 && smem > allowed) {
-        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ, DSC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+template <int NJ, int DS>
+int launch_scan(const DeltaArgs& a, int batch, cudaStream_t stream) {
+    constexpr size_t smem = scan_floats<NJ, DS>() * sizeof(float);
+    static bool raised = false;
+    if (!raised && smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ, DS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
-        allowed = smem;
+        raised = true;
     }
-    // a prompt's scan runs long on few warps: plain stream order, so that its blocks spread evenly over the SMs
-    if (!a.early) return launch_in_order(delta_scan_kernel<NJ, DSC>, grid, dim3(128), smem, stream, a);
-    return launch_pdl(delta_scan_kernel<NJ, DSC>, grid, dim3(128), smem, stream, a);
+    const int vt = 128 / DS;
+    // plain stream order: it runs long on few warps, which are to spread evenly over the SMs
+    return launch_in_order(delta_scan_kernel<NJ, DS>, dim3((a.dv + vt - 1) / vt, a.H, batch), dim3(128), smem, stream, a);
 }
+
+template <int NJ, int DS>
+int launch_step(const DeltaArgs& a, int batch, cudaStream_t stream) {
+    const int vt = 128 / DS;
+    return launch_pdl(delta_step_kernel<NJ, DS>, dim3((a.dv + vt - 1) / vt, a.H, batch), dim3(128), 0, stream, a);
+}
+
+// lanes of a column and float4 a lane for a row of d
+#define BROLM_BY_SIZE(F, ...)                                              \
+    do {                                                                   \
+        if (a.dp <= 32) return F<1, 8>(__VA_ARGS__);                       \
+        if (a.dp <= 64) return F<2, 8>(__VA_ARGS__);                       \
+        if (a.dp <= 128) return F<4, 8>(__VA_ARGS__);                      \
+        if (a.dp <= 256) return F<4, 16>(__VA_ARGS__);                     \
+        return F<8, 16>(__VA_ARGS__);                                      \
+    } while (0)
+
+int check_sizes(const DeltaArgs& a, int batch) {
+    if (a.K < 1 || a.G <= 0 || a.d <= 0 || a.H <= 0 || a.H % a.G || a.dv <= 0) return BROLM_ERR_BAD_SIZE;
+    if (a.H > 65535 || batch > 65535 || a.d > 512) return BROLM_ERR_TOO_LARGE;
+    if (a.state_stride % 4 != 0 || ((uintptr_t)a.state & 15) != 0) return BROLM_ERR_ALIGNMENT;
+    return BROLM_OK;
+}
+
+int step_by_size(const DeltaArgs& a, int batch, cudaStream_t stream) { BROLM_BY_SIZE(launch_step, a, batch, stream); }
+int scan_by_size(const DeltaArgs& a, int batch, cudaStream_t stream) { BROLM_BY_SIZE(launch_scan, a, batch, stream); }
 
 }  // namespace
 
-// proj float [tokens][ldp]: q: G d | k: G d | v: H dv | zb: H | za: H; taps float [K][2 G d + H dv]; the state row holds
-// the K - 1 kept inputs from tail_off on, [K - 1][2 G d + H dv].  u [tokens][ldu], gates [tokens][2 H], qk [tokens][G].
-BROLM_API int brolm_delta_rows(const void* proj, long ldp, const void* taps, int K, int G, int d, int H, int dv,
-                               float norm_eps, float q_scale, const void* a_log, const void* dt_bias, const void* tok_seq,
-                               const void* positions, const void* cu_q, const void* kv_len, const void* slots, void* state,
-                               long state_stride, long tail_off, int move_tail, void* u, long ldu, void* gates, void* qk,
-                               int tokens, cudaStream_t stream) {
-    if (tokens <= 0) return BROLM_OK;
-    if (K < 1 || G <= 0 || d <= 0 || H <= 0 || H % G || dv <= 0) return BROLM_ERR_BAD_SIZE;
-    if (d > 512) return BROLM_ERR_TOO_LARGE;
-    if (((uintptr_t)gates & 7) != 0) return BROLM_ERR_ALIGNMENT;
-    RowsArgs a;
-    a.proj = (const float*)proj; a.ldp = ldp; a.taps = (const float*)taps; a.K = K; a.G = G; a.d = d; a.H = H; a.dv = dv;
+// Floats of one chunk's record of one head.
+BROLM_API int brolm_delta_record() { return REC; }
+
+// One token per sequence.  proj float [tokens][ldp], taps float [K][2 G d + H dv]; the state row of a sequence holds
+// H * dv * round_up(d, 4) floats from `state` on and the ring of kept inputs from tail_off on.  out [tokens][ldo].
+BROLM_API int brolm_delta_step(const void* proj, long ldp, const void* taps, int K, int G, int d, int H, int dv, float norm_eps,
+                               float q_scale, const void* a_log, const void* dt_bias, const void* cu_q, const void* kv_len,
+                               const void* slots, void* state, long state_stride, long tail_off, void* out, long ldo,
+                               int batch, cudaStream_t stream) {
+    if (batch <= 0) return BROLM_OK;
+    DeltaArgs a = {};
+    a.proj = (const float*)proj; a.ldp = ldp; a.taps = (const float*)taps;
+    a.K = K; a.G = G; a.d = d; a.H = H; a.dv = dv; a.dp = (d + 3) & ~3;
     a.norm_eps = norm_eps; a.q_scale = q_scale; a.a_log = (const float*)a_log; a.dt_bias = (const float*)dt_bias;
-    a.tok_seq = (const int32_t*)tok_seq; a.positions = (const int32_t*)positions; a.cu_q = (const int32_t*)cu_q;
-    a.kv_len = (const int32_t*)kv_len; a.slots = (const int32_t*)slots; a.state = (float*)state;
-    a.state_stride = state_stride; a.tail_off = tail_off; a.move_tail = move_tail;
-    a.u = (float*)u; a.ldu = ldu; a.gates = (float*)gates; a.qk = (float*)qk;
-    const int units = G + (H * dv + V_CHUNK - 1) / V_CHUNK + (H + 31) / 32;
-    // few tokens: a unit a warp; many: a block walks a token's units
-    int by = (units + ROWS_WARPS - 1) / ROWS_WARPS;
-    if (by > 65535) by = 65535;
-    dim3 grid(tokens, by);
-    if (d <= 64) return launch_pdl(delta_rows_kernel<2>, grid, dim3(ROWS_WARPS * 32), 0, stream, a);
-    if (d <= 128) return launch_pdl(delta_rows_kernel<4>, grid, dim3(ROWS_WARPS * 32), 0, stream, a);
-    if (d <= 256) return launch_pdl(delta_rows_kernel<8>, grid, dim3(ROWS_WARPS * 32), 0, stream, a);
-    return launch_pdl(delta_rows_kernel<16>, grid, dim3(ROWS_WARPS * 32), 0, stream, a);
+    a.cu_q = (const int32_t*)cu_q; a.kv_len = (const int32_t*)kv_len; a.slots = (const int32_t*)slots;
+    a.state = (float*)state; a.state_stride = state_stride; a.tail_off = tail_off; a.out = (float*)out; a.ldo = ldo;
+    const int bad = check_sizes(a, batch);
+    return bad ? bad : step_by_size(a, batch, stream);
 }
 
-// The state row of a sequence holds H * dv * round_up(d, 4) floats for this recurrence, from `state` on.
-BROLM_API int brolm_delta_scan(const void* u, long ld, const void* gates, const void* qk, int G, int d, int H, int dv,
-                               const void* cu_q, const void* kv_len, const void* slots, void* state, long state_stride,
-                               void* out, long ldo, int batch, int max_q_len, cudaStream_t stream) {
-    if (batch <= 0) return BROLM_OK;
-    if (G <= 0 || d <= 0 || H <= 0 || H % G || dv <= 0) return BROLM_ERR_BAD_SIZE;
-    if (H > 65535 || batch > 65535 || d > 512) return BROLM_ERR_TOO_LARGE;
-    if (state_stride % 4 != 0 || ((uintptr_t)state & 15) != 0) return BROLM_ERR_ALIGNMENT;
-    ScanArgs a;
-    a.u = (const float*)u; a.ld = ld; a.gates = (const float*)gates; a.qk = (const float*)qk;
-    a.G = G; a.H = H; a.d = d; a.dv = dv; a.dp = (d + 3) & ~3;
+// Any number of tokens per sequence, four kernels (three for K = 1).  u [tokens][ldu] (ldu a multiple of four), gates
+// [tokens][2 H] and chunks [tokens / 16 + batch + 1][H][REC] are scratch, 16-byte aligned.
+BROLM_API int brolm_delta_prompt(const void* proj, long ldp, const void* taps, int K, int G, int d, int H, int dv,
+                                 float norm_eps, float q_scale, const void* a_log, const void* dt_bias, const void* tok_seq,
+                                 const void* positions, const void* cu_q, const void* kv_len, const void* slots, void* state,
+                                 long state_stride, long tail_off, void* u, long ldu, void* gates, void* chunks, void* out,
+                                 long ldo, int tokens, int batch, int max_q_len, cudaStream_t stream) {
+    if (batch <= 0 || tokens <= 0) return BROLM_OK;
+    DeltaArgs a = {};
+    a.proj = (const float*)proj; a.ldp = ldp; a.taps = (const float*)taps;
+    a.K = K; a.G = G; a.d = d; a.H = H; a.dv = dv; a.dp = (d + 3) & ~3;
+    a.norm_eps = norm_eps; a.q_scale = q_scale; a.a_log = (const float*)a_log; a.dt_bias = (const float*)dt_bias;
+    a.tok_seq = (const int32_t*)tok_seq; a.positions = (const int32_t*)positions;
     a.cu_q = (const int32_t*)cu_q; a.kv_len = (const int32_t*)kv_len; a.slots = (const int32_t*)slots;
-    a.state = (float*)state; a.state_stride = state_stride; a.out = (float*)out; a.ldo = ldo;
-    a.vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && ((uintptr_t)u & 15) == 0;
-    a.early = max_q_len == 1 ? 1 : 0;
-    const int dp4 = a.dp >> 2, sms = device_sm_count();
-    // a lane keeps nj float4 of a column's states, ds lanes a column; fewer states a lane (more, smaller blocks)
-    // while the grid would leave SMs without a block
-    auto lanes = [&](int nj) { int ds = 1; while (ds * nj < dp4) ds <<= 1; return ds; };
-    auto blocks = [&](int nj) { const int vt = 128 / lanes(nj); return (long long)((dv + vt - 1) / vt) * H * batch; };
-    int nj = 4;
-    while (nj > 1 && lanes(nj) == 1 && nj / 2 >= dp4) nj >>= 1;
-    while (nj > 1 && lanes(nj / 2) <= 32 && blocks(nj) < sms) nj >>= 1;
-    const int ds = lanes(nj);
-    if (ds > 32) return BROLM_ERR_TOO_LARGE;
-    a.ds = ds;
-    const int vt = 128 / ds;
-    const size_t smem = (size_t)2 * SCAN_TC * (2 * a.dp + vt + 4) * sizeof(float);
-    if (smem > 200 * 1024) return BROLM_ERR_TOO_LARGE;
-    dim3 grid((dv + vt - 1) / vt, H, batch);
-    // the sizes of real layers: everything about the row known to the compiler
-    if (a.vec && nj * ds == dp4 && d == a.dp) {
-        if (nj == 1 && ds == 8) return launch_scan_as<1, 8>(a, grid, smem, stream);
-        if (nj == 2 && ds == 8) return launch_scan_as<2, 8>(a, grid, smem, stream);
-        if (nj == 4 && ds == 4) return launch_scan_as<4, 4>(a, grid, smem, stream);
-        if (nj == 4 && ds == 8) return launch_scan_as<4, 8>(a, grid, smem, stream);
-        if (nj == 2 && ds == 16) return launch_scan_as<2, 16>(a, grid, smem, stream);
-        if (nj == 4 && ds == 16) return launch_scan_as<4, 16>(a, grid, smem, stream);
+    a.state = (float*)state; a.state_stride = state_stride; a.tail_off = tail_off;
+    a.u = (float*)u; a.ldu = ldu; a.gates = (float*)gates; a.chunks = (float*)chunks; a.out = (float*)out; a.ldo = ldo;
+    a.tokens = tokens;
+    const int bad = check_sizes(a, batch);
+    if (bad) return bad;
+    if (max_q_len <= 0) return BROLM_ERR_BAD_SIZE;
+    if (ldu % 4 != 0 || (((uintptr_t)u | (uintptr_t)gates | (uintptr_t)chunks) & 15)) return BROLM_ERR_ALIGNMENT;
+    const int C = 2 * G * d + H * dv, v_units = (H * dv + V_CHUNK - 1) / V_CHUNK;
+    a.vec = d % 4 == 0 && dv % 4 == 0;
+    int st;
+    if (a.vec && K <= RUN_TAPS && d <= 256 && ldp % 4 == 0 && tail_off % 4 == 0 &&
+        (((uintptr_t)proj | (uintptr_t)taps) & 15) == 0) {
+        dim3 grid((tokens + RUN - 1) / RUN, (G + v_units + 1 + ROWS_WARPS - 1) / ROWS_WARPS);
+        st = d <= 128 ? launch_pdl(delta_rows_run_kernel<1>, grid, dim3(ROWS_WARPS * 32), 0, stream, a)
+                      : launch_pdl(delta_rows_run_kernel<2>, grid, dim3(ROWS_WARPS * 32), 0, stream, a);
+    } else {
+        int by = (G + v_units + (H + 31) / 32 + ROWS_WARPS - 1) / ROWS_WARPS;
+        if (by > 65535) by = 65535;
+        dim3 grid(tokens, by);
+        st = d <= 64    ? launch_pdl(delta_rows_kernel<2>, grid, dim3(ROWS_WARPS * 32), 0, stream, a)
+             : d <= 128 ? launch_pdl(delta_rows_kernel<4>, grid, dim3(ROWS_WARPS * 32), 0, stream, a)
+             : d <= 256 ? launch_pdl(delta_rows_kernel<8>, grid, dim3(ROWS_WARPS * 32), 0, stream, a)
+                        : launch_pdl(delta_rows_kernel<16>, grid, dim3(ROWS_WARPS * 32), 0, stream, a);
     }
-    if (nj == 1) return launch_scan_as<1, 0>(a, grid, smem, stream);
-    if (nj == 2) return launch_scan_as<2, 0>(a, grid, smem, stream);
-    return launch_scan_as<4, 0>(a, grid, smem, stream);
+    if (st) return st;
+    if (K > 1) {
+        st = launch_pdl(delta_tail_kernel, dim3(batch, (C + 255) / 256), dim3(256), 0, stream, a);
+        if (st) return st;
+    }
+    const size_t smem = (size_t)2 * TC * (a.dp + 4) * sizeof(float);
+    if (smem > 48 * 1024) {
+        static bool raised = false;
+        if (!raised) {
+            const int most = 2 * TC * (512 + 4) * (int)sizeof(float);
+            cudaError_t e = cudaFuncSetAttribute(delta_chunks_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
+            if (e != cudaSuccess) return (int)e;
+            raised = true;
+        }
+    }
+    st = launch_in_order(delta_chunks_kernel, dim3((max_q_len + TC - 1) / TC, H, batch), dim3(128), smem, stream, a);
+    if (st) return st;
+    return scan_by_size(a, batch, stream);
 }

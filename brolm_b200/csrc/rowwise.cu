@@ -130,6 +130,27 @@ __global__ void __launch_bounds__(256) scaled_sum_kernel(const float* __restrict
     out[i] = sa * va + sb * vb;
 }
 
+// The same, four neighbours a thread (n and both strides multiples of four, every row 16-byte aligned).
+__global__ void __launch_bounds__(256) scaled_sum4_kernel(const float* __restrict__ a, int a_parts, long long a_stride, float sa,
+                                                          const float* __restrict__ b, int b_parts, long long b_stride, float sb,
+                                                          float* __restrict__ out, long long n) {
+    pdl_trigger();
+    pdl_wait();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i >= n) return;
+    float4 va = *reinterpret_cast<const float4*>(a + i), vb = *reinterpret_cast<const float4*>(b + i);
+    for (int s = 1; s < a_parts; ++s) {
+        const float4 x = *reinterpret_cast<const float4*>(a + (size_t)s * a_stride + i);
+        va.x += x.x; va.y += x.y; va.z += x.z; va.w += x.w;
+    }
+    for (int s = 1; s < b_parts; ++s) {
+        const float4 x = *reinterpret_cast<const float4*>(b + (size_t)s * b_stride + i);
+        vb.x += x.x; vb.y += x.y; vb.z += x.z; vb.w += x.w;
+    }
+    *reinterpret_cast<float4*>(out + i) = make_float4(sa * va.x + sb * vb.x, sa * va.y + sb * vb.y, sa * va.z + sb * vb.z,
+                                                      sa * va.w + sb * vb.w);
+}
+
 // proj row t: [ q: q_cols | k: k_cols | v: v_cols ] (float or bfloat16).  out row t takes the same layout in O.
 // whole_norm: q <- q * rsqrt(mean(q^2) + eps) * wq over all q_cols at once, the same for k with wk.
 // The cache of this layer is k_pages [page][n_kv][page_size][k_cols / n_kv], v_pages [...][v_cols / n_kv].
@@ -481,6 +502,10 @@ BROLM_API int brolm_scaled_sum(const void* a, int a_parts, long long a_stride, f
                                long long b_stride, float sb, void* out, long long n, cudaStream_t stream) {
     if (n <= 0) return BROLM_OK;
     if (a_parts < 1 || b_parts < 1) return BROLM_ERR_BAD_SIZE;
+    if (n % 4 == 0 && n >= (1 << 18) && (a_parts == 1 || a_stride % 4 == 0) && (b_parts == 1 || b_stride % 4 == 0) &&
+        (((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & 15) == 0)
+        return launch_pdl(scaled_sum4_kernel, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, stream, (const float*)a,
+                          a_parts, a_stride, sa, (const float*)b, b_parts, b_stride, sb, (float*)out, n);
     return launch_pdl(scaled_sum_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const float*)a, a_parts,
                       a_stride, sa, (const float*)b, b_parts, b_stride, sb, (float*)out, n);
 }

@@ -962,52 +962,67 @@ def decay_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int
 
 
 DELTA_NORM_EPS = 1e-6       # under the root of the unit vectors of q and k
+DELTA_CHUNK = 16            # tokens that the recurrence of a prompt takes at a time
 
 
-def delta_rows(proj: torch.Tensor, taps: torch.Tensor, n_kv: int, dim: int, heads: int, v_dim: int, q_scale: float,
-               a_log: torch.Tensor, dt_bias: torch.Tensor, tok_seq: torch.Tensor, positions: torch.Tensor, cu_q: torch.Tensor,
-               kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, tail_off: int, move_tail: bool,
-               u: torch.Tensor, gates: torch.Tensor, qk: torch.Tensor, norm_eps: float = DELTA_NORM_EPS) -> None:
-    """The gated delta rule's inputs from a projection row [q: n_kv * dim | k: n_kv * dim | v: heads * v_dim | heads
-    logits of beta | heads step sizes], all float32: q, k and v after a causal convolution (``taps`` float32 [K, C], row
-    K - 1 the token's own) and silu, q and k as unit vectors per head (q times ``q_scale``), into ``u`` (tokens, C);
-    ``gates`` [tokens, heads, 2] = (decay - 1, beta); ``qk`` [tokens, n_kv] = q . k.  Earlier inputs come from the K - 1
-    rows that ``state[slot, tail_off:]`` keeps; ``move_tail`` (only when every sequence brings one token) moves them on,
-    otherwise ``conv_tail`` does afterwards."""
+def _delta_sizes(proj, taps, n_kv, dim, heads, v_dim, a_log, dt_bias, state, tail_off, out):
     K, C = taps.shape
-    T = proj.shape[0]
     assert C == 2 * n_kv * dim + heads * v_dim and taps.dtype == torch.float32 and taps.is_contiguous()
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= C + 2 * heads
-    assert u.dtype == torch.float32 and u.stride(1) == 1 and u.shape == (T, C) and tail_off + (K - 1) * C <= state.shape[1]
-    assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.numel() == T * heads * 2
-    assert qk.dtype == torch.float32 and qk.is_contiguous() and qk.numel() == T * n_kv
-    assert tok_seq.dtype == torch.int32 and positions.dtype == torch.int32 and positions.numel() == T
+    assert out.dtype == torch.float32 and out.stride(1) == 1 and out.shape == (proj.shape[0], heads * v_dim)
+    assert decay_state_size(heads, dim, v_dim) <= tail_off and tail_off + (K if K > 1 else 0) * C <= state.shape[1]
     for v in (a_log, dt_bias):
         assert v.dtype == torch.float32 and v.is_contiguous() and v.numel() == heads
-    f = _fn("delta_rule", "brolm_delta_rows", [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                               c_long, c_long, c_int, c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p])
-    _check(f(_ptr(proj), proj.stride(0), _ptr(taps), K, n_kv, dim, heads, v_dim, norm_eps, q_scale, _ptr(a_log), _ptr(dt_bias),
-             _ptr(tok_seq), _ptr(positions), *_seq(cu_q, kv_len, slots, state), tail_off, 1 if move_tail else 0, _ptr(u),
-             u.stride(0), _ptr(gates), _ptr(qk), T, _stream()), "delta_rows")
+    return K, C
 
 
-def delta_scan(u: torch.Tensor, gates: torch.Tensor, qk: torch.Tensor, n_kv: int, dim: int, heads: int, v_dim: int,
-               cu_q: torch.Tensor, kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
-               batch: int, max_q_len: int = 0) -> None:
-    """The gated delta rule over the packed tokens, on what ``delta_rows`` made: per head S <- g S, w = beta (v - S^T k),
-    S <- S + k w^T, out = S^T q.  S is the first ``decay_state_size(heads, dim, v_dim)`` floats of ``state[slot]``.
-    ``max_q_len`` 1 says that every sequence brings one token; 0: unknown."""
-    T = u.shape[0]
-    assert u.dtype == torch.float32 and u.stride(1) == 1 and u.shape[1] == 2 * n_kv * dim + heads * v_dim
-    assert gates.dtype == torch.float32 and gates.is_contiguous() and gates.numel() == T * heads * 2
-    assert qk.dtype == torch.float32 and qk.is_contiguous() and qk.numel() == T * n_kv
-    assert out.dtype == torch.float32 and out.stride(1) == 1 and out.shape == (T, heads * v_dim)
-    assert state.shape[1] >= decay_state_size(heads, dim, v_dim)
-    f = _fn("delta_rule", "brolm_delta_scan", [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                                               c_void_p, c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_void_p])
-    _check(f(_ptr(u), u.stride(0), _ptr(gates), _ptr(qk), n_kv, dim, heads, v_dim, *_seq(cu_q, kv_len, slots, state), _ptr(out),
-             out.stride(0), batch, int(max_q_len), _stream()), "delta_scan")
+def delta_step(proj: torch.Tensor, taps: torch.Tensor, n_kv: int, dim: int, heads: int, v_dim: int, a_log: torch.Tensor,
+               dt_bias: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
+               tail_off: int, out: torch.Tensor, batch: int, norm_eps: float = DELTA_NORM_EPS) -> None:
+    """The gated delta rule for one new token per sequence, from the projection to the heads' results, all float32.
+    ``proj`` (tokens, .) = [q: n_kv * dim | k: n_kv * dim | v: heads * v_dim | heads logits of beta | heads step sizes];
+    q, k and v pass a causal convolution (``taps`` [K, C], row K - 1 the token's own) and silu, q and k are made unit
+    vectors per head (q times dim^(-1/2)); then per head S <- g S, w = beta (v - S^T k), S <- S + k w^T, out = S^T q with
+    beta a sigmoid and g = exp(-exp(a_log) softplus(step size + dt_bias)).  ``state[slot]`` holds S
+    (``decay_state_size(heads, dim, v_dim)`` floats) and, from ``tail_off`` on, the newest inputs of the convolution as
+    a ring of K rows (none for K = 1), position p in row p % K."""
+    K, _ = _delta_sizes(proj, taps, n_kv, dim, heads, v_dim, a_log, dt_bias, state, tail_off, out)
+    f = _fn("delta_rule", "brolm_delta_step", [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_long,
+                                               c_void_p, c_long, c_int, c_void_p])
+    _check(f(_ptr(proj), proj.stride(0), _ptr(taps), K, n_kv, dim, heads, v_dim, norm_eps, dim ** -0.5, _ptr(a_log),
+             _ptr(dt_bias), *_seq(cu_q, kv_len, slots, state), tail_off, _ptr(out), out.stride(0), batch, _stream()),
+           "delta_step")
+
+
+def delta_prompt(proj: torch.Tensor, taps: torch.Tensor, n_kv: int, dim: int, heads: int, v_dim: int, a_log: torch.Tensor,
+                 dt_bias: torch.Tensor, tok_seq: torch.Tensor, positions: torch.Tensor, cu_q: torch.Tensor,
+                 kv_len: torch.Tensor, slots: torch.Tensor, state: torch.Tensor, tail_off: int, out: torch.Tensor, batch: int,
+                 max_q_len: int, norm_eps: float = DELTA_NORM_EPS) -> None:
+    """``delta_step`` for any number of tokens per sequence (at most ``max_q_len``): the inputs of the recurrence token by
+    token, the newest ones into the ring, per sixteen tokens what does not hang on the state, then the recurrence."""
+    K, C = _delta_sizes(proj, taps, n_kv, dim, heads, v_dim, a_log, dt_bias, state, tail_off, out)
+    T, dev = proj.shape[0], proj.device
+    assert tok_seq.dtype == torch.int32 and positions.dtype == torch.int32 and positions.numel() == T and max_q_len > 0
+    record = _delta_record()
+    ldu = (C + 3) // 4 * 4
+    u = torch.empty((T, ldu), dtype=torch.float32, device=dev)
+    gates = torch.empty((T, heads, 2), dtype=torch.float32, device=dev)
+    chunks = torch.empty((T // DELTA_CHUNK + batch + 1, heads, record), dtype=torch.float32, device=dev)
+    f = _fn("delta_rule", "brolm_delta_prompt", [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                                 c_void_p, c_long, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
+                                                 c_long, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(proj), proj.stride(0), _ptr(taps), K, n_kv, dim, heads, v_dim, norm_eps, dim ** -0.5, _ptr(a_log),
+             _ptr(dt_bias), _ptr(tok_seq), _ptr(positions), *_seq(cu_q, kv_len, slots, state), tail_off, _ptr(u), ldu,
+             _ptr(gates), _ptr(chunks), _ptr(out), out.stride(0), T, batch, int(max_q_len), _stream()), "delta_prompt")
+    global _launches
+    _launches += 3 if K > 1 else 2      # four kernels, or three
+
+
+def _delta_record() -> int:
+    f = _fn("delta_rule", "brolm_delta_record", [])
+    return int(f())
 
 
 def rotate_heads(rows: torch.Tensor, q_off: int, k_off: int, heads: int, dim: int, positions: torch.Tensor,
@@ -1698,4 +1713,4 @@ __all__ = ["KernelBuildError", "KernelError", "build_all", "launch_count", "devi
            "rope_kv_write", "rope_kv_write_parts", "gated_act", "softcap", "linear_f32", "skinny_gemm", "skinny_qkv_rope", "skinny_ok", "skinny_parts", "skinny_rope_tiles", "gemm_tc", "gemm_tc2", "gemm_tc2_status", "gemm_tc_ok", "gemm_tc_status", "gemm_stream", "gemm_stream_ok", "gemm_stream_parts", "stream_rows",
            "gemm_stream_status", "attention_simt", "attention_prefill_mma", "attention_prefill_tc", "attention_prefill_tc_ok", "attention_prefill_tc_split", "attention_tc_status", "attention_decode_mma",
            "decode_splits", "argmax", "sample", "cast", "bias_act", "scaled_sum", "qkv_norm_write", "gate_group_norm", "head_norm_gate", "rotate_heads",
-           "layernorm", "residual_layernorm", "table_gate", "delta_rows", "delta_scan", "experts_combine", "causal_conv", "conv_tail", "gated_scan", "ssm_scan", "block_matvec_f32", "block_matvec_ok", "split_halves"]
+           "layernorm", "residual_layernorm", "table_gate", "delta_step", "delta_prompt", "experts_combine", "causal_conv", "conv_tail", "gated_scan", "ssm_scan", "block_matvec_f32", "block_matvec_ok", "split_halves"]

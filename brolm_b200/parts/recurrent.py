@@ -306,8 +306,8 @@ class GatedDeltaRule(Part):
 
     Every head's o is divided by its own root mean square, times a gain of ``v_dim`` numbers for all heads (``norm``),
     times silu(W_g x), then W_o.  The projection's sums and everything up to the last product's input are float32 in
-    every mode; S and the convolutions' last taps - 1 inputs are a state row per sequence, zero at the sequence's
-    start."""
+    every mode; S and the convolutions' newest inputs are a state row per sequence, zero at the sequence's start.  A
+    step of single tokens is one kernel from the projection to o; a prompt runs the recurrence sixteen tokens at a time."""
 
     kind = "mixer"
     graph_safe = True
@@ -354,27 +354,24 @@ class GatedDeltaRule(Part):
         self.params = {}
 
     def cache_spec(self):
-        # S, then taps - 1 rows of inputs; a row of the state group is a whole number of 16-byte pieces
-        n = self.tail_off + (self.taps - 1) * self.conv_cols
+        # S, then a ring of inputs; a row of the state group is a whole number of 16-byte pieces
+        n = self.tail_off + (self.taps if self.taps > 1 else 0) * self.conv_cols
         return StateSpec(((n + 3) // 4 * 4,), torch.float32)
 
     def forward(self, x: torch.Tensor, ctx, entry, writes_cache: bool = True) -> torch.Tensor:
         """x (tokens, hidden) -> (tokens, hidden) float32, or partial sums [parts, tokens, hidden]."""
         if not writes_cache:
             raise NotImplementedError("a mixer with a state cannot run on another layer's state")
-        T, dev = x.shape[0], x.device
-        f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
-        seq = (ctx.cu_q, ctx.kv_len, ctx.slots_dev, ctx.state(entry))
-        sizes = (self.kv_heads, self.dim, self.heads, self.v_dim)
-        single = ctx.max_q_len == 1
+        T = x.shape[0]
+        seq = (ctx.cu_q, ctx.kv_len, ctx.slots_dev, ctx.state(entry), self.tail_off)
+        sizes = (self.kv_heads, self.dim, self.heads, self.v_dim, self.a_log, self.dt_bias)
         proj = linear(x, self.w_in, out_dtype=torch.float32)              # [ q | k | v | b | a | gate logits ]
-        u, gates, qk, y = f32(T, self.conv_cols), f32(T, self.heads, 2), f32(T, self.kv_heads), f32(T, self.v_cols)
-        kernels.delta_rows(proj, self.conv, *sizes, self.dim ** -0.5, self.a_log, self.dt_bias, ctx.tok_seq, ctx.positions,
-                           *seq, self.tail_off, single, u, gates, qk)
-        if not single and self.taps > 1:
-            kernels.conv_tail(proj[:, :self.conv_cols], None, self.taps, *seq, self.tail_off, ctx.batch)
-        kernels.delta_scan(u, gates, qk, *sizes, *seq, y, ctx.batch, ctx.max_q_len)
-        out = torch.empty((T, self.v_cols), dtype=ctx.dtype, device=dev)
+        y = torch.empty((T, self.v_cols), dtype=torch.float32, device=x.device)
+        if ctx.max_q_len == 1:
+            kernels.delta_step(proj, self.conv, *sizes, *seq, y, ctx.batch)
+        else:
+            kernels.delta_prompt(proj, self.conv, *sizes, ctx.tok_seq, ctx.positions, *seq, y, ctx.batch, ctx.max_q_len)
+        out = torch.empty((T, self.v_cols), dtype=ctx.dtype, device=x.device)
         kernels.head_norm_gate(y, proj[:, self.gate_from:], self.gain, self.eps, self.heads, "silu", out)
         return linear(out, self.w_o, out_dtype=torch.float32, parts_ok=True)
 

@@ -23,7 +23,8 @@
 //     delta_scan     the recurrence, sixteen tokens at a time.
 // With S0 the state ahead of the sixteen tokens, D(i, j) the product of the decays of tokens j + 1 .. i and D(i) that of
 // the tokens up to i, the recurrence's u solve a triangular system whose matrix needs the keys and gates alone:
-//     u_i + sum_{j < i} beta_i D(i, j) (k_i . k_j) u_j = beta_i (v_i - D(i) S0^T k_i) =: r_i,       u = T r
+//     u_i + sum_{j < i} beta_i D(i, j) (k_i . k_j) u_j = beta_i (v_i - D(i) S0^T k_i),       u = T (..)
+//                                                      = U_i - S0^T w_i,   U = T (beta v),  w = T (beta D k)
 //     o_i = D(i) S0^T q_i + sum_{j <= i} D(i, j) (q_i . k_j) u_j
 //     S   = D(15) S0 + sum_j D(15, j) k_j u_j^T
 // so all products with S0 of the sixteen tokens are independent of one another.  T's entries are at most one in
@@ -72,6 +73,7 @@ struct DeltaArgs {
     float* u;                 // [tokens][ldu]: q | k | v
     long ldu;
     float* gates;             // [tokens][2 H]: (log g, beta) head by head
+    float* w;                 // [tokens][H dp]
     float* chunks;            // [chunk][H][REC]
     float* out;               // [tokens][ldo]; head h at h * dv
     long ldo;
@@ -174,9 +176,9 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) delta_rows_kernel(DeltaArgs a
     }
 }
 
-// The same for up to four taps and sizes in fours: a warp takes its unit of a run of eight packed tokens, four channels
-// a lane and load; the taps' inputs slide through registers, so a token costs one load where the sequence goes on.
-constexpr int RUN = 8, RUN_TAPS = 4;
+// The same for up to four taps and sizes in fours: a warp takes its unit of a run of packed tokens, four channels a lane
+// and load; where the run lies in one sequence all its rows are on their way before the first is used.
+constexpr int RUN = 4, RUN_TAPS = 4;
 
 __device__ __forceinline__ float4 fma4(float4 w, float4 x, float4 c) {
     return make_float4(fmaf(w.x, x.x, c.x), fmaf(w.y, x.y, c.y), fmaf(w.z, x.z, c.z), fmaf(w.w, x.w, c.w));
@@ -190,55 +192,56 @@ __device__ __forceinline__ float4 mul4(float4 a, float f) { return make_float4(a
 // N columns of four channels a lane (col[n] < 0: none), the convolved and activated values handed to `use` per token.
 template <int N, typename F>
 __device__ __forceinline__ void run_of_tokens(const DeltaArgs& a, int C, const int (&col)[N], F use) {
-    const int K = a.K, t0 = blockIdx.x * RUN;
+    const int K = a.K, t0 = blockIdx.x * RUN, n_run = min(RUN, a.tokens - t0);
     const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    float4 w[RUN_TAPS][N], win[RUN_TAPS][N];
+    float4 w[RUN_TAPS][N];
 #pragma unroll
     for (int jj = 0; jj < RUN_TAPS; ++jj)
 #pragma unroll
         for (int n = 0; n < N; ++n) {
             const int j = jj - (RUN_TAPS - K);
             w[jj][n] = j >= 0 && col[n] >= 0 ? *reinterpret_cast<const float4*>(a.taps + (size_t)j * C + col[n]) : zero;
-            win[jj][n] = zero;
         }
-    pdl_wait();
-    int prev_b = -1, prev_pos = -2;
-    for (int i = 0; i < RUN && t0 + i < a.tokens; ++i) {
-        const int t = t0 + i, pos = a.positions[t];
-        if (pos < 0) { prev_b = -1; continue; }
-        const int b = a.tok_seq[t];
-        const bool on = b == prev_b && pos == prev_pos + 1;
-        if (on) {
+    // rows m = 0 .. take tokens t - 3 + m of the sequence that token t (its position pos) belongs to
+    auto fetch = [&](int t, int pos, int b, int m, float4 (&x)[N]) {
+        const int first = a.kv_len[b] - (a.cu_q[b + 1] - a.cu_q[b]), q = pos - (RUN_TAPS - 1) + m;
+        const bool in = q >= 0 && q > pos - K;
+        const float* r = q >= first || !in ? a.proj + (size_t)(in ? t - (RUN_TAPS - 1) + m : t) * a.ldp
+                                           : a.state + (size_t)a.slots[b] * a.state_stride + a.tail_off + (size_t)(q % K) * C;
 #pragma unroll
-            for (int jj = 0; jj < RUN_TAPS - 1; ++jj)
-#pragma unroll
-                for (int n = 0; n < N; ++n) win[jj][n] = win[jj + 1][n];
-        } else {
-            const int q0 = a.cu_q[b], first = a.kv_len[b] - (a.cu_q[b + 1] - q0);
-            const float* ring = a.state + (size_t)a.slots[b] * a.state_stride + a.tail_off;
-#pragma unroll
-            for (int jj = 0; jj < RUN_TAPS - 1; ++jj) {
-                const int q = pos - (RUN_TAPS - 1) + jj;
-                const bool in = q >= 0 && jj >= RUN_TAPS - K;
-                const float* r = q >= first ? a.proj + (size_t)(q0 + q - first) * a.ldp : ring + (size_t)(in ? q % K : 0) * C;
-#pragma unroll
-                for (int n = 0; n < N; ++n) win[jj][n] = in && col[n] >= 0 ? *reinterpret_cast<const float4*>(r + col[n]) : zero;
-            }
-        }
-#pragma unroll
-        for (int n = 0; n < N; ++n)
-            win[RUN_TAPS - 1][n] = col[n] >= 0 ? *reinterpret_cast<const float4*>(a.proj + (size_t)t * a.ldp + col[n]) : zero;
-        prev_b = b;
-        prev_pos = pos;
+        for (int n = 0; n < N; ++n) x[n] = in && col[n] >= 0 ? *reinterpret_cast<const float4*>(r + col[n]) : zero;
+    };
+    auto finish = [&](int t, const float4 (&x0)[N], const float4 (&x1)[N], const float4 (&x2)[N], const float4 (&x3)[N]) {
         float4 v[N];
 #pragma unroll
-        for (int n = 0; n < N; ++n) {
-            v[n] = zero;
-#pragma unroll
-            for (int jj = 0; jj < RUN_TAPS; ++jj) v[n] = fma4(w[jj][n], win[jj][n], v[n]);
-            v[n] = silu4(v[n]);
-        }
+        for (int n = 0; n < N; ++n)
+            v[n] = silu4(fma4(w[3][n], x3[n], fma4(w[2][n], x2[n], fma4(w[1][n], x1[n], fma4(w[0][n], x0[n], zero)))));
         use(t, v);
+    };
+    const int b0 = a.tok_seq[t0], pos0 = a.positions[t0];
+    const bool one = n_run == RUN && pos0 >= 0 && a.tok_seq[t0 + RUN - 1] == b0 && a.positions[t0 + RUN - 1] == pos0 + RUN - 1;
+    pdl_wait();
+    if (one) {
+        float4 x[RUN + RUN_TAPS - 1][N];
+#pragma unroll
+        for (int m = 0; m < RUN_TAPS; ++m) fetch(t0, pos0, b0, m, x[m]);
+#pragma unroll
+        for (int m = RUN_TAPS; m < RUN + RUN_TAPS - 1; ++m)
+#pragma unroll
+            for (int n = 0; n < N; ++n)
+                x[m][n] = col[n] >= 0 ? *reinterpret_cast<const float4*>(a.proj + (size_t)(t0 + m - (RUN_TAPS - 1)) * a.ldp + col[n]) : zero;
+#pragma unroll
+        for (int i = 0; i < RUN; ++i) finish(t0 + i, x[i], x[i + 1], x[i + 2], x[i + 3]);
+        return;
+    }
+    for (int i = 0; i < n_run; ++i) {
+        const int t = t0 + i, pos = a.positions[t];
+        if (pos < 0) continue;
+        const int b = a.tok_seq[t];
+        float4 x[RUN_TAPS][N];
+#pragma unroll
+        for (int m = 0; m < RUN_TAPS; ++m) fetch(t, pos, b, m, x[m]);
+        finish(t, x[0], x[1], x[2], x[3]);
     }
 }
 
@@ -437,19 +440,21 @@ __global__ void __launch_bounds__(128) delta_step_kernel(DeltaArgs a) {
 }
 
 // ---------------------------------------------------------------------------
-// delta_chunks: a block takes sixteen tokens of one (sequence, head) and leaves a record of REC floats:
-//   T [16][20], B [16][20] (rows padded against bank conflicts), B_ij = D(i, j) (q_i . k_j) for j <= i,
-//   beta [16], beta_i D(i) [16], D(i) [16], D(15, i) [16], expm1(log D(15)), three unused.
-// Tokens beyond the sequence's end have k = q = 0, log g = 0 and beta = 0, and change nothing.
+// delta_chunks: a block takes sixteen tokens of one (sequence, head).  It writes w (rows of dp, zeros beyond d), puts U in
+// v's place and leaves a record of REC floats:
+//   B [16][20] (rows padded against bank conflicts), B_ij = D(i, j) (q_i . k_j) for j <= i,
+//   D(i) [16], D(15, i) [16], expm1(log D(15)), three unused.
+// Tokens beyond the sequence's end have k = q = v = 0, log g = 0 and beta = 0, and change nothing.
 // Record number of chunk c of sequence b: cu_q[b] / 16 + b + c (sequences never share one).
 // ---------------------------------------------------------------------------
-constexpr int TC = 16, MR = 20, OFF_B = TC * MR, OFF_V = 2 * TC * MR, REC = OFF_V + 4 * TC + 4;
+constexpr int TC = 16, MR = 20, OFF_V = TC * MR, REC = OFF_V + 2 * TC + 4;
 
 __device__ __forceinline__ int record_of(int q0, int b, int chunk) { return q0 / TC + b + chunk; }
 
 __global__ void __launch_bounds__(128) delta_chunks_kernel(DeltaArgs a) {
     extern __shared__ __align__(16) float sm[];            // k [16][ld], q [16][ld]
     __shared__ float lg[TC], be[TC], A[TC][TC + 1];
+    __shared__ __align__(16) float Tb[TC][MR], Tk[TC][MR]; // T beta and T beta D
     const int chunk = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
     const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0, t0 = chunk * TC;
     if (a.kv_len[b] <= 0 || t0 >= q_len) return;
@@ -504,19 +509,18 @@ __global__ void __launch_bounds__(128) delta_chunks_kernel(DeltaArgs a) {
         for (int l = j + 1; l <= i; ++l) s += lg[l];
         const float D = i >= j ? expf(s) : 0.0f;
         A[i][j] = i > j ? be[i] * D * kk[m] : 0.0f;
-        rec[OFF_B + i * MR + j] = D * qk[m];
-        if (i == TC - 1) rec[OFF_V + 3 * TC + j] = D;
+        rec[i * MR + j] = D * qk[m];
+        if (i == TC - 1) rec[OFF_V + TC + j] = D;
         if (j == 0) {
-            const float s_all = s + lg[0], all = expf(s_all);
-            rec[OFF_V + i] = be[i];
-            rec[OFF_V + TC + i] = be[i] * all;
-            rec[OFF_V + 2 * TC + i] = all;
-            if (i == TC - 1) rec[OFF_V + 4 * TC] = expm1f(s_all);
+            rec[OFF_V + i] = expf(s + lg[0]);
+            if (i == TC - 1) rec[OFF_V + 2 * TC] = expm1f(s + lg[0]);
         }
     }
     __syncthreads();
     if (tid < TC) {                                        // column tid of T, from the diagonal down
-        float x[TC];
+        float x[TC], s_all = 0.0f;
+        for (int l = 0; l <= tid; ++l) s_all += lg[l];
+        const float fb = be[tid], fk = fb * expf(s_all);
 #pragma unroll
         for (int r = 0; r < TC; ++r) {
             float s = 0.0f;
@@ -525,13 +529,41 @@ __global__ void __launch_bounds__(128) delta_chunks_kernel(DeltaArgs a) {
             x[r] = r < tid ? 0.0f : r == tid ? 1.0f : -s;
         }
 #pragma unroll
-        for (int r = 0; r < TC; ++r) rec[r * MR + tid] = x[r];
+        for (int r = 0; r < TC; ++r) {
+            Tb[r][tid] = x[r] * fb;
+            Tk[r][tid] = x[r] * fk;
+        }
+    }
+    __syncthreads();
+    // a column of k, or of v, a thread: sixteen sums over the sixteen tokens
+    for (int c = tid; c < a.dp + a.dv; c += 128) {
+        const bool is_k = c < a.dp;
+        const int cv = c - a.dp;
+        float* vcol = a.u + (size_t)(q0 + t0) * a.ldu + 2 * a.G * a.d + h * a.dv + cv;
+        float x[TC];
+#pragma unroll
+        for (int j = 0; j < TC; ++j) x[j] = is_k ? sk[j * ld + c] : (j < n_tok ? vcol[(size_t)j * a.ldu] : 0.0f);
+        float* dst = is_k ? a.w + (size_t)(q0 + t0) * a.H * a.dp + h * a.dp + c : vcol;
+        const size_t step = is_k ? (size_t)a.H * a.dp : (size_t)a.ldu;
+        const float* m = is_k ? &Tk[0][0] : &Tb[0][0];
+#pragma unroll
+        for (int r = 0; r < TC; ++r) {
+            float y = 0.0f;
+#pragma unroll
+            for (int j = 0; j <= r; ++j) y = fmaf(m[r * MR + j], x[j], y);
+            if (r < n_tok) dst[(size_t)r * step] = y;
+        }
     }
 }
 
 // ---------------------------------------------------------------------------
-// delta_scan: blocks and lanes as in delta_step; sixteen tokens and their record at a time, three stages of cp.async.
-// A warp works on its own columns alone.  Of a column's sixteen sums lane ds ends up with those of tokens ds, ds + DS, ..
+// delta_scan: a block of 128 threads takes one (sequence, head) and sixteen value columns, sixteen tokens at a time.  A
+// warp holds a quarter of d for all sixteen columns, a lane NJ x 4 entries of d (f = (warp NJ + j) 8 + lane mod 8 counts
+// fours of d) for four columns: a number read from shared memory (which hands out 32 a cycle) meets four states.
+//   1. partial products of w and q with the state, folded across the eight lanes of a column group, left per warp;
+//   2. the four warps' parts joined: u = U - S0^T w (warps 0 and 1), D S0^T q (warps 2 and 3);
+//   3. the state's update by all, o by warps 2 and 3.
+// The rows come through three stages of cp.async.
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void cp4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -540,55 +572,68 @@ __device__ __forceinline__ void cp16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-constexpr int STAGES = 3, XR = 20;                         // XR: floats between two columns' sixteen exchanged numbers
+constexpr int VC = 16;                                     // value columns of a block
+constexpr int PR = 20;                                     // floats between two rows of sixteen columns
+// w, q, k rows [16][DP], U [16][PR], the record
+template <int NJ> __host__ __device__ constexpr int scan_stage() { return 3 * TC * 128 * NJ + TC * PR + REC; }
+template <int NJ> __host__ __device__ constexpr int scan_stages() { return NJ == 4 ? 2 : 3; }
+template <int NJ> __host__ __device__ constexpr int scan_floats() {
+    return scan_stages<NJ>() * scan_stage<NJ>() + 4 * 2 * TC * PR + 2 * TC * PR;
+}
 
-template <int NJ, int DS> __host__ __device__ constexpr int scan_stage() { return TC * (2 * 4 * NJ * DS + 128 / DS) + REC; }
-template <int NJ, int DS> __host__ __device__ constexpr int scan_floats() { return STAGES * scan_stage<NJ, DS>() + 2 * (128 / DS) * XR; }
-
-template <int NJ, int DS>
+template <int NJ>
 __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
     extern __shared__ __align__(16) float sm[];
-    constexpr int DP = 4 * NJ * DS, VT = 128 / DS, NT = TC / DS, STAGE = scan_stage<NJ, DS>();
-    const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VT;
+    constexpr int DP = 128 * NJ, STAGE = scan_stage<NJ>(), STAGES = scan_stages<NJ>();
+    const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VC;
     const int kv_len = a.kv_len[b];
     if (kv_len <= 0) return;
     const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0;
     if (q_len <= 0) return;
-    const int hk = h / (a.H / a.G), tid = threadIdx.x;
-    const int ds = tid % DS, vcol = tid / DS, v = v0 + vcol;
-    const bool live = v < a.dv;
-    const int dp4 = a.dp >> 2;
-    float* st = a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + (live ? v : 0)) * a.dp;
-    float* xr = sm + STAGES * STAGE + vcol * XR;           // the column's exchanged r, then u
-    float* xu = xr + VT * XR;
-    f32x2 S[2 * NJ];
+    const int hk = h / (a.H / a.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int ds = lane & 7, cg = lane >> 3;               // place in d, group of four columns
+    const int dp4 = a.dp >> 2, vt = min(VC, a.dv - v0);
+    float* part = sm + STAGES * STAGE;                     // [4 warps][32 rows][PR]
+    float* us = part + 4 * 2 * TC * PR;                    // [16][PR] u
+    float* ud = us + TC * PR;                              // [16][PR] D(15, j) u_j
+    f32x2 S[NJ][4][2];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-        const int f = j * DS + ds;
-        float4 s4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (live && f < dp4) s4 = *reinterpret_cast<const float4*>(st + 4 * f);
-        S[2 * j] = pack2(s4.x, s4.y);
-        S[2 * j + 1] = pack2(s4.z, s4.w);
+        const int f = (warp * NJ + j) * 8 + ds;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const int v = 4 * cg + c;
+            float4 s4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (v < vt && f < dp4)
+                s4 = *reinterpret_cast<const float4*>(a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + v0 + v) * a.dp + 4 * f);
+            S[j][c][0] = pack2(s4.x, s4.y);
+            S[j][c][1] = pack2(s4.z, s4.w);
+        }
     }
-    const int n_chunks = (q_len + TC - 1) / TC, vt_here = min(VT, a.dv - v0);
+    const int n_chunks = (q_len + TC - 1) / TC;
     // rows padded to DP, value columns beyond dv and tokens beyond the end read as zeros
-    if (DP != a.d || vt_here != VT || (q_len & (TC - 1))) {
+    if (DP != a.d || vt != VC || (q_len & (TC - 1))) {
         for (int i = tid; i < STAGES * STAGE; i += 128) sm[i] = 0.0f;
         __syncthreads();
     }
     const int q_off = hk * a.d, k_off = a.G * a.d + hk * a.d, v_off = 2 * a.G * a.d + h * a.dv + v0;
     auto issue = [&](int chunk) {
-        float* sk = sm + (chunk % STAGES) * STAGE;
-        float* sq = sk + TC * DP;
-        float* sv = sq + TC * DP;
-        float* sr = sv + TC * VT;
+        float* sw = sm + (chunk % STAGES) * STAGE;
+        float* sq = sw + TC * DP;
+        float* sk = sq + TC * DP;
+        float* sv = sk + TC * DP;
         const int t0 = chunk * TC, n_tok = min(TC, q_len - t0);
         if (n_tok < TC && chunk >= STAGES) {               // the last stage holds older tokens where there are none now
-            for (int i = tid; i < (TC - n_tok) * DP; i += 128) sk[n_tok * DP + i] = sq[n_tok * DP + i] = 0.0f;
-            for (int i = tid; i < (TC - n_tok) * VT; i += 128) sv[n_tok * VT + i] = 0.0f;
+            for (int i = tid; i < (TC - n_tok) * DP; i += 128)
+                sw[n_tok * DP + i] = sq[n_tok * DP + i] = sk[n_tok * DP + i] = 0.0f;
+            for (int i = tid; i < (TC - n_tok) * PR; i += 128) sv[n_tok * PR + i] = 0.0f;
+        }
+        for (int idx = tid; idx < n_tok * dp4; idx += 128) {
+            const int tt = idx / dp4, c = (idx - tt * dp4) << 2;
+            cp16(sw + tt * DP + c, a.w + (size_t)(q0 + t0 + tt) * a.H * a.dp + h * a.dp + c);
         }
         if (a.vec) {
-            const int d4 = a.d >> 2, v4 = vt_here >> 2;
+            const int d4 = a.d >> 2, v4 = vt >> 2;
             for (int idx = tid; idx < n_tok * d4; idx += 128) {
                 const int tt = idx / d4, c = (idx - tt * d4) << 2;
                 const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ldu + c;
@@ -597,7 +642,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
             }
             for (int idx = tid; idx < n_tok * v4; idx += 128) {
                 const int tt = idx / v4, c = (idx - tt * v4) << 2;
-                cp16(sv + tt * VT + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
+                cp16(sv + tt * PR + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
             }
         } else {
             for (int idx = tid; idx < n_tok * a.d; idx += 128) {
@@ -606,143 +651,165 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
                 cp4(sq + tt * DP + c, row + q_off);
                 cp4(sk + tt * DP + c, row + k_off);
             }
-            for (int idx = tid; idx < n_tok * vt_here; idx += 128) {
-                const int tt = idx / vt_here, c = idx - tt * vt_here;
-                cp4(sv + tt * VT + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
+            for (int idx = tid; idx < n_tok * vt; idx += 128) {
+                const int tt = idx / vt, c = idx - tt * vt;
+                cp4(sv + tt * PR + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
             }
         }
         const float* rec = a.chunks + ((size_t)record_of(q0, b, chunk) * a.H + h) * REC;
-        for (int idx = tid; idx < REC / 4; idx += 128) cp16(sr + 4 * idx, rec + 4 * idx);
+        for (int idx = tid; idx < REC / 4; idx += 128) cp16(sv + TC * PR + 4 * idx, rec + 4 * idx);
     };
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s) {
         if (s < n_chunks) issue(s);
         asm volatile("cp.async.commit_group;" ::: "memory");
     }
+    const int jrow = tid >> 2, jcg = tid & 3;              // phase 2: row (of 32) and group of four columns
+    const bool out4 = vt == VC && a.dv % 4 == 0 && a.ldo % 4 == 0 && ((uintptr_t)a.out & 15) == 0;
     for (int kc = 0; kc < n_chunks; ++kc) {
         asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
         __syncthreads();                                   // this stage has landed, and no warp works on the one before
         if (kc + STAGES - 1 < n_chunks) issue(kc + STAGES - 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        const float* sk = sm + (kc % STAGES) * STAGE;
-        const float* sq = sk + TC * DP;
-        const float* sv = sq + TC * DP;
-        const float* sr = sv + TC * VT;
-        // sixteen sums over the column's d, folded across its lanes: at every step a lane hands half of what it holds to
-        // the lane `o` away and adds what it gets to the half it keeps; p is the token ds + DS (p mod NT) of lane p / NT
-        auto sums = [&](const float* rows, float (&mine)[NT]) {
-            float s[TC];
+        const float* sw = sm + (kc % STAGES) * STAGE;      // w rows, q rows behind them
+        const float* sk = sw + 2 * TC * DP;
+        const float* sv = sk + TC * DP;
+        const float* sr = sv + TC * PR;
 #pragma unroll
-            for (int p = 0; p < TC; ++p) {
-                const int tok = p / NT + DS * (p % NT);
-                const ulonglong2* r = reinterpret_cast<const ulonglong2*>(rows + tok * DP) + ds;
-                f32x2 acc = 0ull, acc1 = 0ull;
+        for (int g = 0; g < 4; ++g) {                      // eight rows at a time; lane ds ends up with row ds of them
+            float s[8][4];
+#pragma unroll
+            for (int r = 0; r < 8; ++r) {
+                f32x2 acc[4] = {0ull, 0ull, 0ull, 0ull};
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
-                    const ulonglong2 x = r[j * DS];
-                    acc = fma2(S[2 * j], x.x, acc);
-                    acc1 = fma2(S[2 * j + 1], x.y, acc1);
-                }
-                const float2 e = unpack2(acc), f = unpack2(acc1);
-                s[p] = (e.x + e.y) + (f.x + f.y);
-            }
+                    const ulonglong2 x = reinterpret_cast<const ulonglong2*>(sw + (8 * g + r) * DP)[(warp * NJ + j) * 8 + ds];
 #pragma unroll
-            for (int n = TC / 2, o = DS / 2; o > 0; n >>= 1, o >>= 1) {
+                    for (int c = 0; c < 4; ++c) acc[c] = fma2(S[j][c][1], x.y, fma2(S[j][c][0], x.x, acc[c]));
+                }
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    const float2 e = unpack2(acc[c]);
+                    s[r][c] = e.x + e.y;
+                }
+            }
+            // at every step a lane hands half of the rows it holds to the lane `o` away and adds what it gets to the rest
+#pragma unroll
+            for (int n = 4, o = 4; o > 0; n >>= 1, o >>= 1) {
                 const bool up = (ds & o) != 0;
 #pragma unroll
-                for (int i = 0; i < TC / 2; ++i)
-                    if (i < n) {
-                        const float send = up ? s[i] : s[i + n], keep = up ? s[i + n] : s[i];
-                        s[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                for (int r = 0; r < 4; ++r)
+                    if (r < n) {
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) {
+                            const float send = up ? s[r][c] : s[r + n][c], keep = up ? s[r + n][c] : s[r][c];
+                            s[r][c] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
                     }
             }
-#pragma unroll
-            for (int i = 0; i < NT; ++i) mine[i] = s[i];
-        };
-        float pk[NT], pq[NT];
-        sums(sk, pk);
-#pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            const int tok = ds + DS * i;
-            xr[tok] = fmaf(-sr[OFF_V + TC + tok], pk[i], sr[OFF_V + tok] * sv[tok * VT + vcol]);
+            *reinterpret_cast<float4*>(part + (warp * 2 * TC + 8 * g + ds) * PR + 4 * cg) = make_float4(s[0][0], s[0][1], s[0][2], s[0][3]);
         }
-        sums(sq, pq);
-        __syncwarp();
-        float u[TC];
+        __syncthreads();
+        float4 y = *reinterpret_cast<const float4*>(part + jrow * PR + 4 * jcg);
 #pragma unroll
-        for (int j = 0; j < TC; j += 4) {
-            const float4 x = *reinterpret_cast<const float4*>(xr + j);
-            u[j] = x.x; u[j + 1] = x.y; u[j + 2] = x.z; u[j + 3] = x.w;
+        for (int w = 1; w < 4; ++w) {
+            const float4 x = *reinterpret_cast<const float4*>(part + (w * 2 * TC + jrow) * PR + 4 * jcg);
+            y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w;
+        }
+        const int tok = jrow & (TC - 1);
+        if (jrow < TC) {
+            const float4 U = *reinterpret_cast<const float4*>(sv + tok * PR + 4 * jcg);
+            const float f = sr[OFF_V + TC + tok];
+            y = make_float4(U.x - y.x, U.y - y.y, U.z - y.z, U.w - y.w);
+            *reinterpret_cast<float4*>(us + tok * PR + 4 * jcg) = y;
+            *reinterpret_cast<float4*>(ud + tok * PR + 4 * jcg) = mul4(y, f);
+        }
+        __syncthreads();
+        const float dm1 = sr[OFF_V + 2 * TC];
+        float st[NJ][4][4];
+#pragma unroll
+        for (int j = 0; j < NJ; ++j)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const float2 e = unpack2(S[j][c][0]), f = unpack2(S[j][c][1]);
+                st[j][c][0] = fmaf(dm1, e.x, e.x);
+                st[j][c][1] = fmaf(dm1, e.y, e.y);
+                st[j][c][2] = fmaf(dm1, f.x, f.x);
+                st[j][c][3] = fmaf(dm1, f.y, f.y);
+            }
+#pragma unroll
+        for (int t = 0; t < TC; ++t) {
+            const float4 u4 = *reinterpret_cast<const float4*>(ud + t * PR + 4 * cg);
+            const float uu[4] = {u4.x, u4.y, u4.z, u4.w};
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+                const float4 k = *reinterpret_cast<const float4*>(sk + t * DP + 4 * ((warp * NJ + j) * 8 + ds));
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    st[j][c][0] = fmaf(k.x, uu[c], st[j][c][0]);
+                    st[j][c][1] = fmaf(k.y, uu[c], st[j][c][1]);
+                    st[j][c][2] = fmaf(k.z, uu[c], st[j][c][2]);
+                    st[j][c][3] = fmaf(k.w, uu[c], st[j][c][3]);
+                }
+            }
         }
 #pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            const int tok = ds + DS * i;
-            float s = 0.0f, s1 = 0.0f;
+        for (int j = 0; j < NJ; ++j)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                S[j][c][0] = pack2(st[j][c][0], st[j][c][1]);
+                S[j][c][1] = pack2(st[j][c][2], st[j][c][3]);
+            }
+        const int t = kc * TC + tok;
+        if (jrow >= TC && t < q_len) {
+            y = mul4(y, sr[OFF_V + tok]);
 #pragma unroll
             for (int j = 0; j < TC; j += 4) {
                 const float4 m = *reinterpret_cast<const float4*>(sr + tok * MR + j);
-                s = fmaf(m.x, u[j], fmaf(m.y, u[j + 1], s));
-                s1 = fmaf(m.z, u[j + 2], fmaf(m.w, u[j + 3], s1));
+                const float mm[4] = {m.x, m.y, m.z, m.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float4 u4 = *reinterpret_cast<const float4*>(us + (j + e) * PR + 4 * jcg);
+                    y = fma4(make_float4(mm[e], mm[e], mm[e], mm[e]), u4, y);
+                }
             }
-            xu[tok] = s + s1;
-        }
-        __syncwarp();
+            float* o = a.out + (size_t)(q0 + t) * a.ldo + (size_t)h * a.dv + v0 + 4 * jcg;
+            if (out4) {
+                *reinterpret_cast<float4*>(o) = y;
+            } else {
+                const float e[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
-        for (int j = 0; j < TC; j += 4) {
-            const float4 x = *reinterpret_cast<const float4*>(xu + j);
-            u[j] = x.x; u[j + 1] = x.y; u[j + 2] = x.z; u[j + 3] = x.w;
-        }
-#pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            const int tok = ds + DS * i, t = kc * TC + tok;
-            float s = sr[OFF_V + 2 * TC + tok] * pq[i], s1 = 0.0f;
-#pragma unroll
-            for (int j = 0; j < TC; j += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(sr + OFF_B + tok * MR + j);
-                s = fmaf(m.x, u[j], fmaf(m.y, u[j + 1], s));
-                s1 = fmaf(m.z, u[j + 2], fmaf(m.w, u[j + 3], s1));
-            }
-            if (live && t < q_len) a.out[(size_t)(q0 + t) * a.ldo + (size_t)h * a.dv + v] = s + s1;
-        }
-        const float dm1 = sr[OFF_V + 4 * TC];
-        const f32x2 dm2 = pack2(dm1, dm1);
-#pragma unroll
-        for (int j = 0; j < 2 * NJ; ++j) S[j] = fma2(dm2, S[j], S[j]);
-#pragma unroll
-        for (int tok = 0; tok < TC; ++tok) {
-            const float f = sr[OFF_V + 3 * TC + tok] * u[tok];
-            const f32x2 f2 = pack2(f, f);
-            const ulonglong2* r = reinterpret_cast<const ulonglong2*>(sk + tok * DP) + ds;
-#pragma unroll
-            for (int j = 0; j < NJ; ++j) {
-                const ulonglong2 x = r[j * DS];
-                S[2 * j] = fma2(x.x, f2, S[2 * j]);
-                S[2 * j + 1] = fma2(x.y, f2, S[2 * j + 1]);
+                for (int c = 0; c < 4; ++c)
+                    if (4 * jcg + c < vt) o[c] = e[c];
             }
         }
     }
-    if (live) {
 #pragma unroll
-        for (int j = 0; j < NJ; ++j) {
-            const int f = j * DS + ds;
-            const float2 e = unpack2(S[2 * j]), g = unpack2(S[2 * j + 1]);
-            if (f < dp4) *reinterpret_cast<float4*>(st + 4 * f) = make_float4(e.x, e.y, g.x, g.y);
+    for (int j = 0; j < NJ; ++j) {
+        const int f = (warp * NJ + j) * 8 + ds;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const int v = 4 * cg + c;
+            const float2 e = unpack2(S[j][c][0]), g = unpack2(S[j][c][1]);
+            if (v < vt && f < dp4)
+                *reinterpret_cast<float4*>(a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + v0 + v) * a.dp + 4 * f) =
+                    make_float4(e.x, e.y, g.x, g.y);
         }
     }
 }
 
-template <int NJ, int DS>
+template <int NJ>
 int launch_scan(const DeltaArgs& a, int batch, cudaStream_t stream) {
-    constexpr size_t smem = scan_floats<NJ, DS>() * sizeof(float);
+    constexpr size_t smem = scan_floats<NJ>() * sizeof(float);
+    static_assert(smem <= 227 * 1024, "the stages do not fit an SM");
     static bool raised = false;
-    if (!raised && smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ, DS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (!raised) {
+        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         raised = true;
     }
-    const int vt = 128 / DS;
     // plain stream order: it runs long on few warps, which are to spread evenly over the SMs
-    return launch_in_order(delta_scan_kernel<NJ, DS>, dim3((a.dv + vt - 1) / vt, a.H, batch), dim3(128), smem, stream, a);
+    return launch_in_order(delta_scan_kernel<NJ>, dim3((a.dv + VC - 1) / VC, a.H, batch), dim3(128), smem, stream, a);
 }
 
 template <int NJ, int DS>
@@ -751,16 +818,6 @@ int launch_step(const DeltaArgs& a, int batch, cudaStream_t stream) {
     return launch_pdl(delta_step_kernel<NJ, DS>, dim3((a.dv + vt - 1) / vt, a.H, batch), dim3(128), 0, stream, a);
 }
 
-// lanes of a column and float4 a lane for a row of d
-#define BROLM_BY_SIZE(F, ...)                                              \
-    do {                                                                   \
-        if (a.dp <= 32) return F<1, 8>(__VA_ARGS__);                       \
-        if (a.dp <= 64) return F<2, 8>(__VA_ARGS__);                       \
-        if (a.dp <= 128) return F<4, 8>(__VA_ARGS__);                      \
-        if (a.dp <= 256) return F<4, 16>(__VA_ARGS__);                     \
-        return F<8, 16>(__VA_ARGS__);                                      \
-    } while (0)
-
 int check_sizes(const DeltaArgs& a, int batch) {
     if (a.K < 1 || a.G <= 0 || a.d <= 0 || a.H <= 0 || a.H % a.G || a.dv <= 0) return BROLM_ERR_BAD_SIZE;
     if (a.H > 65535 || batch > 65535 || a.d > 512) return BROLM_ERR_TOO_LARGE;
@@ -768,8 +825,19 @@ int check_sizes(const DeltaArgs& a, int batch) {
     return BROLM_OK;
 }
 
-int step_by_size(const DeltaArgs& a, int batch, cudaStream_t stream) { BROLM_BY_SIZE(launch_step, a, batch, stream); }
-int scan_by_size(const DeltaArgs& a, int batch, cudaStream_t stream) { BROLM_BY_SIZE(launch_scan, a, batch, stream); }
+// lanes of a column and float4 a lane for a row of d
+int step_by_size(const DeltaArgs& a, int batch, cudaStream_t stream) {
+    if (a.dp <= 32) return launch_step<1, 8>(a, batch, stream);
+    if (a.dp <= 64) return launch_step<2, 8>(a, batch, stream);
+    if (a.dp <= 128) return launch_step<4, 8>(a, batch, stream);
+    if (a.dp <= 256) return launch_step<4, 16>(a, batch, stream);
+    return launch_step<8, 16>(a, batch, stream);
+}
+int scan_by_size(const DeltaArgs& a, int batch, cudaStream_t stream) {
+    if (a.dp <= 128) return launch_scan<1>(a, batch, stream);
+    if (a.dp <= 256) return launch_scan<2>(a, batch, stream);
+    return launch_scan<4>(a, batch, stream);
+}
 
 }  // namespace
 
@@ -794,11 +862,11 @@ BROLM_API int brolm_delta_step(const void* proj, long ldp, const void* taps, int
 }
 
 // Any number of tokens per sequence, four kernels (three for K = 1).  u [tokens][ldu] (ldu a multiple of four), gates
-// [tokens][2 H] and chunks [tokens / 16 + batch + 1][H][REC] are scratch, 16-byte aligned.
+// [tokens][2 H], w [tokens][H * round_up(d, 4)] and chunks [tokens / 16 + batch + 1][H][REC] are scratch, 16-byte aligned.
 BROLM_API int brolm_delta_prompt(const void* proj, long ldp, const void* taps, int K, int G, int d, int H, int dv,
                                  float norm_eps, float q_scale, const void* a_log, const void* dt_bias, const void* tok_seq,
                                  const void* positions, const void* cu_q, const void* kv_len, const void* slots, void* state,
-                                 long state_stride, long tail_off, void* u, long ldu, void* gates, void* chunks, void* out,
+                                 long state_stride, long tail_off, void* u, long ldu, void* gates, void* w, void* chunks, void* out,
                                  long ldo, int tokens, int batch, int max_q_len, cudaStream_t stream) {
     if (batch <= 0 || tokens <= 0) return BROLM_OK;
     DeltaArgs a = {};
@@ -808,12 +876,12 @@ BROLM_API int brolm_delta_prompt(const void* proj, long ldp, const void* taps, i
     a.tok_seq = (const int32_t*)tok_seq; a.positions = (const int32_t*)positions;
     a.cu_q = (const int32_t*)cu_q; a.kv_len = (const int32_t*)kv_len; a.slots = (const int32_t*)slots;
     a.state = (float*)state; a.state_stride = state_stride; a.tail_off = tail_off;
-    a.u = (float*)u; a.ldu = ldu; a.gates = (float*)gates; a.chunks = (float*)chunks; a.out = (float*)out; a.ldo = ldo;
+    a.u = (float*)u; a.ldu = ldu; a.gates = (float*)gates; a.w = (float*)w; a.chunks = (float*)chunks; a.out = (float*)out; a.ldo = ldo;
     a.tokens = tokens;
     const int bad = check_sizes(a, batch);
     if (bad) return bad;
     if (max_q_len <= 0) return BROLM_ERR_BAD_SIZE;
-    if (ldu % 4 != 0 || (((uintptr_t)u | (uintptr_t)gates | (uintptr_t)chunks) & 15)) return BROLM_ERR_ALIGNMENT;
+    if (ldu % 4 != 0 || (((uintptr_t)u | (uintptr_t)gates | (uintptr_t)w | (uintptr_t)chunks) & 15)) return BROLM_ERR_ALIGNMENT;
     const int C = 2 * G * d + H * dv, v_units = (H * dv + V_CHUNK - 1) / V_CHUNK;
     a.vec = d % 4 == 0 && dv % 4 == 0;
     int st;

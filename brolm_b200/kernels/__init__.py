@@ -1008,14 +1008,15 @@ def delta_prompt(proj: torch.Tensor, taps: torch.Tensor, n_kv: int, dim: int, he
     ldu = (C + 3) // 4 * 4
     u = torch.empty((T, ldu), dtype=torch.float32, device=dev)
     gates = torch.empty((T, heads, 2), dtype=torch.float32, device=dev)
+    w = torch.empty((T, heads * ((dim + 3) // 4 * 4)), dtype=torch.float32, device=dev)
     chunks = torch.empty((T // DELTA_CHUNK + batch + 1, heads, record), dtype=torch.float32, device=dev)
     f = _fn("delta_rule", "brolm_delta_prompt", [c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                                                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                                  c_void_p, c_long, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p,
-                                                 c_long, c_int, c_int, c_int, c_void_p])
+                                                 c_void_p, c_long, c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(proj), proj.stride(0), _ptr(taps), K, n_kv, dim, heads, v_dim, norm_eps, dim ** -0.5, _ptr(a_log),
              _ptr(dt_bias), _ptr(tok_seq), _ptr(positions), *_seq(cu_q, kv_len, slots, state), tail_off, _ptr(u), ldu,
-             _ptr(gates), _ptr(chunks), _ptr(out), out.stride(0), T, batch, int(max_q_len), _stream()), "delta_prompt")
+             _ptr(gates), _ptr(w), _ptr(chunks), _ptr(out), out.stride(0), T, batch, int(max_q_len), _stream()), "delta_prompt")
     global _launches
     _launches += 3 if K > 1 else 2      # four kernels, or three
 

@@ -557,12 +557,12 @@ __global__ void __launch_bounds__(128) delta_chunks_kernel(DeltaArgs a) {
 }
 
 // ---------------------------------------------------------------------------
-// delta_scan: a block of 128 threads takes one (sequence, head) and sixteen value columns, sixteen tokens at a time.  A
-// warp holds a quarter of d for all sixteen columns, a lane NJ x 4 entries of d (f = (warp NJ + j) 8 + lane mod 8 counts
-// fours of d) for four columns: a number read from shared memory (which hands out 32 a cycle) meets four states.
-//   1. partial products of w and q with the state, folded across the eight lanes of a column group, left per warp;
-//   2. the four warps' parts joined: u = U - S0^T w (warps 0 and 1), D S0^T q (warps 2 and 3);
-//   3. the state's update by all, o by warps 2 and 3.
+// delta_scan: a block of 256 threads takes one (sequence, head) and sixteen value columns, sixteen tokens at a time.  A
+// warp holds an eighth of d for all sixteen columns, a lane NJ x 4 entries of d (f = (warp NJ + j) 4 + lane mod 4 counts
+// fours of d) for two columns.  With two warps a scheduler one issues while the other waits.
+//   1. partial products of w and q with the state, folded across the four lanes of a column pair, left per warp;
+//   2. the eight warps' parts joined: u = U - S0^T w (warps 0 to 3), D S0^T q (warps 4 to 7);
+//   3. the state's update by all, o by warps 4 to 7.
 // The rows come through three stages of cp.async.
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void cp4(float* dst, const float* src) {
@@ -577,12 +577,14 @@ constexpr int PR = 20;                                     // floats between two
 // w, q, k rows [16][DP], U [16][PR], the record
 template <int NJ> __host__ __device__ constexpr int scan_stage() { return 3 * TC * 128 * NJ + TC * PR + REC; }
 template <int NJ> __host__ __device__ constexpr int scan_stages() { return NJ == 4 ? 2 : 3; }
+constexpr int SCAN_WARPS = 8, SCAN_THREADS = 32 * SCAN_WARPS;
 template <int NJ> __host__ __device__ constexpr int scan_floats() {
-    return scan_stages<NJ>() * scan_stage<NJ>() + 4 * 2 * TC * PR + 2 * TC * PR;
+    return scan_stages<NJ>() * scan_stage<NJ>() + SCAN_WARPS * 2 * TC * PR + 2 * TC * PR;
 }
 
-template <int NJ>
-__global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
+// EXACT: d is DP, every row is copied in fours and all sixteen columns are there: the copies' indices are shifts.
+template <int NJ, bool EXACT>
+__global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(DeltaArgs a) {
     extern __shared__ __align__(16) float sm[];
     constexpr int DP = 128 * NJ, STAGE = scan_stage<NJ>(), STAGES = scan_stages<NJ>();
     const int b = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * VC;
@@ -591,18 +593,18 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
     const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0;
     if (q_len <= 0) return;
     const int hk = h / (a.H / a.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int ds = lane & 7, cg = lane >> 3;               // place in d, group of four columns
-    const int dp4 = a.dp >> 2, vt = min(VC, a.dv - v0);
-    float* part = sm + STAGES * STAGE;                     // [4 warps][32 rows][PR]
-    float* us = part + 4 * 2 * TC * PR;                    // [16][PR] u
+    const int ds = lane & 3, cg = lane >> 2;               // place in d, pair of columns
+    const int dp4 = EXACT ? DP / 4 : a.dp >> 2, vt = EXACT ? VC : min(VC, a.dv - v0);
+    float* part = sm + STAGES * STAGE;                     // [8 warps][32 rows][PR]
+    float* us = part + SCAN_WARPS * 2 * TC * PR;                 // [16][PR] u
     float* ud = us + TC * PR;                              // [16][PR] D(15, j) u_j
-    f32x2 S[NJ][4][2];
+    f32x2 S[NJ][2][2];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-        const int f = (warp * NJ + j) * 8 + ds;
+        const int f = (warp * NJ + j) * 4 + ds;
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            const int v = 4 * cg + c;
+        for (int c = 0; c < 2; ++c) {
+            const int v = 2 * cg + c;
             float4 s4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (v < vt && f < dp4)
                 s4 = *reinterpret_cast<const float4*>(a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + v0 + v) * a.dp + 4 * f);
@@ -612,8 +614,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
     }
     const int n_chunks = (q_len + TC - 1) / TC;
     // rows padded to DP, value columns beyond dv and tokens beyond the end read as zeros
-    if (DP != a.d || vt != VC || (q_len & (TC - 1))) {
-        for (int i = tid; i < STAGES * STAGE; i += 128) sm[i] = 0.0f;
+    if (!EXACT || (q_len & (TC - 1))) {
+        for (int i = tid; i < STAGES * STAGE; i += SCAN_THREADS) sm[i] = 0.0f;
         __syncthreads();
     }
     const int q_off = hk * a.d, k_off = a.G * a.d + hk * a.d, v_off = 2 * a.G * a.d + h * a.dv + v0;
@@ -624,48 +626,48 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
         float* sv = sk + TC * DP;
         const int t0 = chunk * TC, n_tok = min(TC, q_len - t0);
         if (n_tok < TC && chunk >= STAGES) {               // the last stage holds older tokens where there are none now
-            for (int i = tid; i < (TC - n_tok) * DP; i += 128)
+            for (int i = tid; i < (TC - n_tok) * DP; i += SCAN_THREADS)
                 sw[n_tok * DP + i] = sq[n_tok * DP + i] = sk[n_tok * DP + i] = 0.0f;
-            for (int i = tid; i < (TC - n_tok) * PR; i += 128) sv[n_tok * PR + i] = 0.0f;
+            for (int i = tid; i < (TC - n_tok) * PR; i += SCAN_THREADS) sv[n_tok * PR + i] = 0.0f;
         }
-        for (int idx = tid; idx < n_tok * dp4; idx += 128) {
+        for (int idx = tid; idx < n_tok * dp4; idx += SCAN_THREADS) {
             const int tt = idx / dp4, c = (idx - tt * dp4) << 2;
             cp16(sw + tt * DP + c, a.w + (size_t)(q0 + t0 + tt) * a.H * a.dp + h * a.dp + c);
         }
-        if (a.vec) {
-            const int d4 = a.d >> 2, v4 = vt >> 2;
-            for (int idx = tid; idx < n_tok * d4; idx += 128) {
+        if (EXACT || a.vec) {
+            const int d4 = EXACT ? DP / 4 : a.d >> 2, v4 = vt >> 2;
+            for (int idx = tid; idx < n_tok * d4; idx += SCAN_THREADS) {
                 const int tt = idx / d4, c = (idx - tt * d4) << 2;
                 const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ldu + c;
                 cp16(sq + tt * DP + c, row + q_off);
                 cp16(sk + tt * DP + c, row + k_off);
             }
-            for (int idx = tid; idx < n_tok * v4; idx += 128) {
+            for (int idx = tid; idx < n_tok * v4; idx += SCAN_THREADS) {
                 const int tt = idx / v4, c = (idx - tt * v4) << 2;
                 cp16(sv + tt * PR + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
             }
         } else {
-            for (int idx = tid; idx < n_tok * a.d; idx += 128) {
+            for (int idx = tid; idx < n_tok * a.d; idx += SCAN_THREADS) {
                 const int tt = idx / a.d, c = idx - tt * a.d;
                 const float* row = a.u + (size_t)(q0 + t0 + tt) * a.ldu + c;
                 cp4(sq + tt * DP + c, row + q_off);
                 cp4(sk + tt * DP + c, row + k_off);
             }
-            for (int idx = tid; idx < n_tok * vt; idx += 128) {
+            for (int idx = tid; idx < n_tok * vt; idx += SCAN_THREADS) {
                 const int tt = idx / vt, c = idx - tt * vt;
                 cp4(sv + tt * PR + c, a.u + (size_t)(q0 + t0 + tt) * a.ldu + v_off + c);
             }
         }
         const float* rec = a.chunks + ((size_t)record_of(q0, b, chunk) * a.H + h) * REC;
-        for (int idx = tid; idx < REC / 4; idx += 128) cp16(sv + TC * PR + 4 * idx, rec + 4 * idx);
+        for (int idx = tid; idx < REC / 4; idx += SCAN_THREADS) cp16(sv + TC * PR + 4 * idx, rec + 4 * idx);
     };
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s) {
         if (s < n_chunks) issue(s);
         asm volatile("cp.async.commit_group;" ::: "memory");
     }
-    const int jrow = tid >> 2, jcg = tid & 3;              // phase 2: row (of 32) and group of four columns
-    const bool out4 = vt == VC && a.dv % 4 == 0 && a.ldo % 4 == 0 && ((uintptr_t)a.out & 15) == 0;
+    const int jrow = tid >> 3, jcg = tid & 7;              // phase 2: row (of 32) and pair of columns
+    const bool out2 = vt == VC && a.dv % 2 == 0 && a.ldo % 2 == 0 && ((uintptr_t)a.out & 7) == 0;
     for (int kc = 0; kc < n_chunks; ++kc) {
         asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
         __syncthreads();                                   // this stage has landed, and no warp works on the one before
@@ -676,61 +678,66 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
         const float* sv = sk + TC * DP;
         const float* sr = sv + TC * PR;
 #pragma unroll
-        for (int g = 0; g < 4; ++g) {                      // eight rows at a time; lane ds ends up with row ds of them
-            float s[8][4];
+        for (int g = 0; g < 4; ++g) {                      // eight rows at a time; lane ds ends up with rows 2 ds, 2 ds + 1
+            float s[8][2];
 #pragma unroll
             for (int r = 0; r < 8; ++r) {
-                f32x2 acc[4] = {0ull, 0ull, 0ull, 0ull};
+                f32x2 acc[2][2] = {{0ull, 0ull}, {0ull, 0ull}};
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
-                    const ulonglong2 x = reinterpret_cast<const ulonglong2*>(sw + (8 * g + r) * DP)[(warp * NJ + j) * 8 + ds];
+                    const ulonglong2 x = reinterpret_cast<const ulonglong2*>(sw + (8 * g + r) * DP)[(warp * NJ + j) * 4 + ds];
 #pragma unroll
-                    for (int c = 0; c < 4; ++c) acc[c] = fma2(S[j][c][1], x.y, fma2(S[j][c][0], x.x, acc[c]));
+                    for (int c = 0; c < 2; ++c) {
+                        acc[c][0] = fma2(S[j][c][0], x.x, acc[c][0]);
+                        acc[c][1] = fma2(S[j][c][1], x.y, acc[c][1]);
+                    }
                 }
 #pragma unroll
-                for (int c = 0; c < 4; ++c) {
-                    const float2 e = unpack2(acc[c]);
-                    s[r][c] = e.x + e.y;
+                for (int c = 0; c < 2; ++c) {
+                    const float2 e = unpack2(acc[c][0]), f = unpack2(acc[c][1]);
+                    s[r][c] = (e.x + e.y) + (f.x + f.y);
                 }
             }
             // at every step a lane hands half of the rows it holds to the lane `o` away and adds what it gets to the rest
 #pragma unroll
-            for (int n = 4, o = 4; o > 0; n >>= 1, o >>= 1) {
+            for (int n = 4, o = 2; o > 0; n >>= 1, o >>= 1) {
                 const bool up = (ds & o) != 0;
 #pragma unroll
                 for (int r = 0; r < 4; ++r)
                     if (r < n) {
 #pragma unroll
-                        for (int c = 0; c < 4; ++c) {
+                        for (int c = 0; c < 2; ++c) {
                             const float send = up ? s[r][c] : s[r + n][c], keep = up ? s[r + n][c] : s[r][c];
                             s[r][c] = keep + __shfl_xor_sync(0xffffffffu, send, o);
                         }
                     }
             }
-            *reinterpret_cast<float4*>(part + (warp * 2 * TC + 8 * g + ds) * PR + 4 * cg) = make_float4(s[0][0], s[0][1], s[0][2], s[0][3]);
+#pragma unroll
+            for (int r = 0; r < 2; ++r)
+                *reinterpret_cast<float2*>(part + (warp * 2 * TC + 8 * g + 2 * ds + r) * PR + 2 * cg) = make_float2(s[r][0], s[r][1]);
         }
         __syncthreads();
-        float4 y = *reinterpret_cast<const float4*>(part + jrow * PR + 4 * jcg);
+        float2 y = make_float2(0.0f, 0.0f);
 #pragma unroll
-        for (int w = 1; w < 4; ++w) {
-            const float4 x = *reinterpret_cast<const float4*>(part + (w * 2 * TC + jrow) * PR + 4 * jcg);
-            y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w;
+        for (int w = 0; w < SCAN_WARPS; ++w) {
+            const float2 x = *reinterpret_cast<const float2*>(part + (w * 2 * TC + jrow) * PR + 2 * jcg);
+            y.x += x.x; y.y += x.y;
         }
         const int tok = jrow & (TC - 1);
         if (jrow < TC) {
-            const float4 U = *reinterpret_cast<const float4*>(sv + tok * PR + 4 * jcg);
+            const float2 U = *reinterpret_cast<const float2*>(sv + tok * PR + 2 * jcg);
             const float f = sr[OFF_V + TC + tok];
-            y = make_float4(U.x - y.x, U.y - y.y, U.z - y.z, U.w - y.w);
-            *reinterpret_cast<float4*>(us + tok * PR + 4 * jcg) = y;
-            *reinterpret_cast<float4*>(ud + tok * PR + 4 * jcg) = mul4(y, f);
+            y = make_float2(U.x - y.x, U.y - y.y);
+            *reinterpret_cast<float2*>(us + tok * PR + 2 * jcg) = y;
+            *reinterpret_cast<float2*>(ud + tok * PR + 2 * jcg) = make_float2(y.x * f, y.y * f);
         }
         __syncthreads();
         const float dm1 = sr[OFF_V + 2 * TC];
-        float st[NJ][4][4];
+        float st[NJ][2][4];
 #pragma unroll
         for (int j = 0; j < NJ; ++j)
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
+            for (int c = 0; c < 2; ++c) {
                 const float2 e = unpack2(S[j][c][0]), f = unpack2(S[j][c][1]);
                 st[j][c][0] = fmaf(dm1, e.x, e.x);
                 st[j][c][1] = fmaf(dm1, e.y, e.y);
@@ -739,13 +746,13 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
             }
 #pragma unroll
         for (int t = 0; t < TC; ++t) {
-            const float4 u4 = *reinterpret_cast<const float4*>(ud + t * PR + 4 * cg);
-            const float uu[4] = {u4.x, u4.y, u4.z, u4.w};
+            const float2 u2 = *reinterpret_cast<const float2*>(ud + t * PR + 2 * cg);
+            const float uu[2] = {u2.x, u2.y};
 #pragma unroll
             for (int j = 0; j < NJ; ++j) {
-                const float4 k = *reinterpret_cast<const float4*>(sk + t * DP + 4 * ((warp * NJ + j) * 8 + ds));
+                const float4 k = *reinterpret_cast<const float4*>(sk + t * DP + 4 * ((warp * NJ + j) * 4 + ds));
 #pragma unroll
-                for (int c = 0; c < 4; ++c) {
+                for (int c = 0; c < 2; ++c) {
                     st[j][c][0] = fmaf(k.x, uu[c], st[j][c][0]);
                     st[j][c][1] = fmaf(k.y, uu[c], st[j][c][1]);
                     st[j][c][2] = fmaf(k.z, uu[c], st[j][c][2]);
@@ -756,40 +763,40 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
 #pragma unroll
         for (int j = 0; j < NJ; ++j)
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
+            for (int c = 0; c < 2; ++c) {
                 S[j][c][0] = pack2(st[j][c][0], st[j][c][1]);
                 S[j][c][1] = pack2(st[j][c][2], st[j][c][3]);
             }
         const int t = kc * TC + tok;
         if (jrow >= TC && t < q_len) {
-            y = mul4(y, sr[OFF_V + tok]);
+            const float f = sr[OFF_V + tok];
+            y.x *= f; y.y *= f;
 #pragma unroll
             for (int j = 0; j < TC; j += 4) {
                 const float4 m = *reinterpret_cast<const float4*>(sr + tok * MR + j);
                 const float mm[4] = {m.x, m.y, m.z, m.w};
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float4 u4 = *reinterpret_cast<const float4*>(us + (j + e) * PR + 4 * jcg);
-                    y = fma4(make_float4(mm[e], mm[e], mm[e], mm[e]), u4, y);
+                    const float2 u2 = *reinterpret_cast<const float2*>(us + (j + e) * PR + 2 * jcg);
+                    y.x = fmaf(mm[e], u2.x, y.x);
+                    y.y = fmaf(mm[e], u2.y, y.y);
                 }
             }
-            float* o = a.out + (size_t)(q0 + t) * a.ldo + (size_t)h * a.dv + v0 + 4 * jcg;
-            if (out4) {
-                *reinterpret_cast<float4*>(o) = y;
+            float* o = a.out + (size_t)(q0 + t) * a.ldo + (size_t)h * a.dv + v0 + 2 * jcg;
+            if (out2) {
+                *reinterpret_cast<float2*>(o) = y;
             } else {
-                const float e[4] = {y.x, y.y, y.z, y.w};
-#pragma unroll
-                for (int c = 0; c < 4; ++c)
-                    if (4 * jcg + c < vt) o[c] = e[c];
+                if (2 * jcg < vt) o[0] = y.x;
+                if (2 * jcg + 1 < vt) o[1] = y.y;
             }
         }
     }
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-        const int f = (warp * NJ + j) * 8 + ds;
+        const int f = (warp * NJ + j) * 4 + ds;
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            const int v = 4 * cg + c;
+        for (int c = 0; c < 2; ++c) {
+            const int v = 2 * cg + c;
             const float2 e = unpack2(S[j][c][0]), g = unpack2(S[j][c][1]);
             if (v < vt && f < dp4)
                 *reinterpret_cast<float4*>(a.state + (size_t)a.slots[b] * a.state_stride + ((size_t)h * a.dv + v0 + v) * a.dp + 4 * f) =
@@ -798,18 +805,24 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a) {
     }
 }
 
-template <int NJ>
-int launch_scan(const DeltaArgs& a, int batch, cudaStream_t stream) {
+template <int NJ, bool EXACT>
+int launch_scan_as(const DeltaArgs& a, int batch, cudaStream_t stream) {
     constexpr size_t smem = scan_floats<NJ>() * sizeof(float);
     static_assert(smem <= 227 * 1024, "the stages do not fit an SM");
     static bool raised = false;
     if (!raised) {
-        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NJ, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         raised = true;
     }
     // plain stream order: it runs long on few warps, which are to spread evenly over the SMs
-    return launch_in_order(delta_scan_kernel<NJ>, dim3((a.dv + VC - 1) / VC, a.H, batch), dim3(128), smem, stream, a);
+    return launch_in_order(delta_scan_kernel<NJ, EXACT>, dim3((a.dv + VC - 1) / VC, a.H, batch), dim3(SCAN_THREADS), smem, stream, a);
+}
+
+template <int NJ>
+int launch_scan(const DeltaArgs& a, int batch, cudaStream_t stream) {
+    return a.vec && a.d == 128 * NJ && a.dv % VC == 0 ? launch_scan_as<NJ, true>(a, batch, stream)
+                                                      : launch_scan_as<NJ, false>(a, batch, stream);
 }
 
 template <int NJ, int DS>

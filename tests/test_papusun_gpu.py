@@ -36,6 +36,8 @@ def setups(tmp_path_factory):
         if dtype == "bfloat16":
             errs = plain.rounding_errors(config, weights, random_prompts(config["vocab"], [9, 64, 150, 300], seed=21))
             ROUNDING[name] = (errs[int(0.9 * (len(errs) - 1))], errs[-1])
+        if dtype == "float32":
+            FLOAT[name] = max(TOL["float32"], 4 * own_float_error(config, weights))
         out[(name, dtype)] = (folder, config, weights, bb.load_model(folder, dtype=dtype, device=DEV))
     return out
 
@@ -45,6 +47,23 @@ def rel(got, ref):
     return float((got.double().cpu() - ref).abs().max()) / max(float(ref.abs().max()), 1e-3)
 
 
+def own_float_error(config, weights):
+    """The largest error the plain implementation itself makes in float32 on the requests of these tests: a result that is
+    divided by its own root mean square and happens to be small leaves some positions with fewer digits than others."""
+    worst = 0.0
+    for seed, lens in ((13, [1, 140, 17, 66, 130]), (19, [420]), (14, [300])):
+        for p in random_prompts(config["vocab"], lens, seed):
+            ref = plain.forward(config, weights, p)
+            plain.F64 = torch.float32
+            try:
+                own = plain.forward(config, weights, p).double()
+            finally:
+                plain.F64 = torch.float64
+            worst = max(worst, float((own - ref).abs().max() / ref.abs().max()))
+    return worst
+
+
+FLOAT: dict = {}        # name -> the bar of a float32 row (filled by the fixture)
 # name -> (nine rows in ten, all rows) of the error that rounding alone makes on the oracle (filled by the fixture)
 ROUNDING: dict = {}
 
@@ -57,7 +76,9 @@ def check(got, ref, dtype, what, name):
     ref = ref.double()
     rows = (got.double().cpu() - ref).abs().reshape(-1, ref.shape[-1]).amax(dim=1) / max(float(ref.abs().max()), 1e-3)
     if dtype == "float32":
-        assert float(rows.max()) <= TOL[dtype], f"{what}: relative error {float(rows.max()):.3e} exceeds {TOL[dtype]:.0e}"
+        assert float(rows.max()) <= FLOAT[name], f"{what}: relative error {float(rows.max()):.3e} exceeds {FLOAT[name]:.0e}"
+        # (what is wrong for a reason other than rounding is wrong at more than a row in ten)
+        assert float(rows.sort().values[int(0.9 * (len(rows) - 1))]) <= TOL[dtype], what
         return
     q90 = float(rows.sort().values[int(0.9 * (len(rows) - 1))])
     most, worst = ROUNDING[name]
@@ -158,7 +179,7 @@ def test_unequal_batches_against_each_alone(setups, name, dtype):
             check(together[i], refs[i], dtype, f"request {i} in batch {ids}", name)
             single = run(alone, [i])[i]
             # what else is in the batch changes nothing beyond rounding
-            assert rel(together[i], single.cpu()) <= (1e-5 if dtype == "float32" else 2 * TOL[dtype])
+            assert rel(together[i], single.cpu()) <= (FLOAT[name] if dtype == "float32" else 2 * TOL[dtype])
     assert eng.cache.live_slots == 0 and all(g.pool.held_pages == 0 for g in eng.cache.kv_groups)
 
 

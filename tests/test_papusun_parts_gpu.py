@@ -35,7 +35,7 @@ def test_layer_norm_alone_and_behind_the_sum(W, wd):
     g = torch.Generator().manual_seed(W)
     T, parts = 5, 3
     h = torch.randn(T, W, generator=g) + 3.0                   # a mean well off zero
-    h[1] = 1e-3 * torch.randn(W, generator=g) + 100.0          # a spread next to the eps, far from zero
+    h[1] = 1e-2 * torch.randn(W, generator=g) + 100.0          # a spread not far above the eps, a mean far from zero
     h[2] = 0.25                                                # no spread at all
     y = torch.randn(parts, T, W, generator=g)
     y[:, 1:3] *= 1e-4
@@ -47,7 +47,7 @@ def test_layer_norm_alone_and_behind_the_sum(W, wd):
     ref = lambda x: plain.layer_norm(x.double(), w.double(), eps)
     out = norm.apply(h.to(DEV), torch.float32)
     close(out[[0, 3, 4]], ref(h)[[0, 3, 4]], what="alone")
-    close(out[1], ref(h)[1], what="far from zero", tol=5e-3)   # (the row itself has two digits of its spread left)
+    close(out[1], ref(h)[1], what="far from zero", tol=2e-3)   # (a float has three digits left for such a row's spread)
     assert float(out[2].abs().max()) <= 1e-2
     close(norm.apply(h.to(DEV), torch.bfloat16, rows=i32(4, 0)), ref(h)[[4, 0]], torch.bfloat16, "picked rows")
     total = y.double().sum(dim=0)
@@ -141,8 +141,9 @@ def test_delta_rule_remembers_for_thousands_of_tokens():
     case = DeltaCase(G, d, H, dv, K, T, seed=9)
     g = torch.Generator().manual_seed(10)
     proj = case.proj
+    case.taps.fill_(1.0)
+    case.taps_dev = case.taps.to(DEV)
     axes = torch.full((T, d), -30.0)                           # silu(-30) is next to nothing: unit vectors along one axis
-    axes[:, :] = -30.0
     pick = 1 + torch.randint(0, d - 1, (T,), generator=g)
     pick[0] = 0
     axes[torch.arange(T), pick] = 5.0

@@ -47,8 +47,9 @@ struct NormArgs {
 };
 
 // C > 0: the row in registers, four neighbours a thread and chunk of 1024; C = 0: any width, plain loops.
-template <typename W, typename O, int C>
-__global__ void __launch_bounds__(256, C <= 2 ? 4 : C <= 4 ? 3 : 1) layernorm_kernel(NormArgs a) {
+// ONE: y in one part (a prompt): without the room for several parts' loads more blocks share an SM.
+template <typename W, typename O, int C, bool ONE>
+__global__ void __launch_bounds__(256, ONE ? (C <= 2 ? 6 : C <= 4 ? 4 : 2) : (C <= 2 ? 4 : C <= 4 ? 3 : 1)) layernorm_kernel(NormArgs a) {
     __shared__ float scratch[64];
     const int r = blockIdx.x, hidden = a.hidden;
     const float inv_n = 1.0f / (float)hidden;
@@ -111,7 +112,9 @@ __global__ void __launch_bounds__(256, C <= 2 ? 4 : C <= 4 ? 3 : 1) layernorm_ke
             for (int c = 0; c < C; ++c) {
                 const int i = (c * 256 + threadIdx.x) * 4;
                 v[c][0] = v[c][1] = v[c][2] = v[c][3] = 0.0f;
-                if (i < hidden) {
+                if constexpr (ONE) {
+                    if (i < hidden) load4(yr + i, v[c]);
+                } else if (i < hidden) {
                     constexpr int AT_ONCE = 4;       // slices whose loads go out together
                     for (int s0 = 0; s0 < a.n_parts; s0 += AT_ONCE) {
                         float t[AT_ONCE][4];
@@ -187,12 +190,16 @@ int launch_norm(const NormArgs& a, int n, cudaStream_t s) {
     int c = 0;
     if (a.hidden % 4 == 0 && !(bits & 15) && a.part_stride % 4 == 0)
         c = a.hidden <= 1024 ? 1 : a.hidden <= 2048 ? 2 : a.hidden <= 3072 ? 3 : a.hidden <= 4096 ? 4 : a.hidden <= 8192 ? 8 : 0;
-    if (c == 1) return launch_pdl(layernorm_kernel<W, O, 1>, dim3(n), dim3(256), 0, s, a);
-    if (c == 2) return launch_pdl(layernorm_kernel<W, O, 2>, dim3(n), dim3(256), 0, s, a);
-    if (c == 3) return launch_pdl(layernorm_kernel<W, O, 3>, dim3(n), dim3(256), 0, s, a);
-    if (c == 4) return launch_pdl(layernorm_kernel<W, O, 4>, dim3(n), dim3(256), 0, s, a);
-    if (c == 8) return launch_pdl(layernorm_kernel<W, O, 8>, dim3(n), dim3(256), 0, s, a);
-    return launch_pdl(layernorm_kernel<W, O, 0>, dim3(n), dim3(256), 0, s, a);
+    const bool one = a.n_parts <= 1;
+#define BROLM_LN(C) return one ? launch_pdl(layernorm_kernel<W, O, C, true>, dim3(n), dim3(256), 0, s, a) \
+                               : launch_pdl(layernorm_kernel<W, O, C, false>, dim3(n), dim3(256), 0, s, a)
+    if (c == 1) BROLM_LN(1);
+    if (c == 2) BROLM_LN(2);
+    if (c == 3) BROLM_LN(3);
+    if (c == 4) BROLM_LN(4);
+    if (c == 8) BROLM_LN(8);
+#undef BROLM_LN
+    return launch_pdl(layernorm_kernel<W, O, 0, false>, dim3(n), dim3(256), 0, s, a);
 }
 
 int launch_any(const NormArgs& a, int w_dtype, int out_dtype, int n, cudaStream_t s) {

@@ -830,7 +830,7 @@ def papusun_main(args, pk) -> int:
     layers = [dict(type="parallel", mixer=pair, mlp=mlp), dict(type="latent_attention", mixer=lat, mlp=mlp),
               dict(type="parallel", mixer=pair, mlp=mlp), dict(type="latent_attention", mixer=dict(lat, kv_from=1), mlp=mlp)]
     xcfg = bb.PapusunConfig.from_dict(dict(architecture="Papusun", vocab=z["vocab"], width=W, layers=layers, norm=dict(eps=1e-5),
-                                           token_side=dict(dim=z["side"]), logit_scale=0.5))
+                                           token_side=dict(dim=z["side"]), logit_scale=0.25))
     cmlp = dict(kind="dense", ff=ff * 3 // 2)
     cattn = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=d ** -0.5, softcap=30.0, bias_max=128, bias_rows=32)
     light = dict(heads=DH, dim=dd, vdim=ddv, decay=[1.0 - 2.0 ** (-3.0 - 7.0 * h / max(DH - 1, 1)) for h in range(DH)])

@@ -66,7 +66,7 @@ CFG_T = model(51, 40, 1e-6, 5, 0.3, [
 # U: sizes the tensor-core kernels take (value heads of the key heads' size and of another), windows of a whole number of
 # pages and one more, a reader whose window is narrower, q/k heads of the recurrence as long as a row of lanes and longer.
 CFG_U = model(64, 64, 1e-5, 16, 2.0, [
-    parallel(left(4, 4, 32, 32, 0.18, 25.0, rot(1000.0, 32, (4.0, 1.0, 4.0, 128))), right(2, 1, 128, 32, 4), 0.8, 0.9, ff=64),
+    parallel(left(4, 4, 32, 32, 0.18, 25.0, rot(1000.0, 32, (5.0, 1.0, 4.0, 128))), right(2, 1, 128, 32, 4), 0.8, 0.9, ff=64),
     latent(4, 16, 16, 32, 32, 48, 0.2, 128, 10000.0, ff=128),
     parallel(left(4, 1, 32, 48, 0.2, 10.0, rot(10000.0, 16)), right(2, 2, 136, 16, 4), 1.25, 1.0, ff=64),
     latent(8, 32, 16, 16, 64, 48, 0.15, 65, 10000.0, kv_from=1, ff=64),

@@ -19,8 +19,8 @@ pytestmark = pytest.mark.gpu
 
 def draw_left(rng, tensor_sizes):
     kv = rng.choice([1, 2, 3])
-    d = rng.choice([16, 32, 64, 96] if tensor_sizes else [4, 6, 8, 16, 20, 32, 64])
-    dv = rng.choice([d, d, 16, 48, 80, 192] if tensor_sizes else [d, 3, 4, 12, 32, 80])
+    d = rng.choice([16, 32, 64, 80] if tensor_sizes else [4, 6, 8, 16, 20, 32, 64])
+    dv = rng.choice([d, d, 16, 48, 112, 176] if tensor_sizes else [d, 3, 4, 12, 32, 80])
     scaling = rng.choice([None, (2.0, 1.0, 4.0, 16), (8.0, 1.0, 4.0, 64), (40.0, 2.0, 7.0, 128), (3.0, 1.5, 1.5, 32)])
     return left(kv * rng.choice([1, 2, 4]), kv, d, dv, rng.choice([0.1, 0.3, 1.0]), rng.choice([0.0, 5.0, 30.0]),
                 rot(rng.choice([100.0, 10000.0]), 2 * rng.randint(1, d // 2), scaling))
